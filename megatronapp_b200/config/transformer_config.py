@@ -311,8 +311,8 @@ class TransformerConfig(ModelParallelConfig):
         if self.cp_comm_type is not None and isinstance(self.cp_comm_type, list):
             if len(self.cp_comm_type) != self.num_layers:
                 raise ValueError("cp_comm_type list must have num_layers entries")
-        if self.moe_router_group_score not in ("topk_sum", "max"):
-            raise ValueError("moe_router_group_score must be topk_sum | max")
+        if self.moe_router_group_score not in ("topk_sum", "max", "top2_sum"):
+            raise ValueError("moe_router_group_score must be topk_sum | max | top2_sum")
         if self.kernel_backend not in ("auto", "b200", "torch"):
             raise ValueError("kernel_backend must be auto | b200 | torch")
 

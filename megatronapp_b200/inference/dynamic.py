@@ -12,8 +12,9 @@ request's slots (padded over requests), so admission, retirement and preemption 
 
 Layers need not be softmax attention with their own K/V.  Latent-attention layers page one latent vector per token
 (``attend_latent``), and a layer may read the pages another layer wrote; ``attend_mixed`` serves attention whose
-softmax weights are mixed across heads, ``attend_window`` sliding-window attention with a distance penalty and a sink.  Recurrent mixers keep a fixed-size state per
-request instead of pages: every request owns a *state row* for its lifetime (``recurrent_state`` hands out per-layer
+softmax weights are mixed across heads, ``attend_window`` sliding-window attention with a distance penalty and a sink,
+``attend_sigmoid`` attention with logistic weights; ``kv_pages`` / ``latent_pages`` and ``write_slots`` let a layer's kernel put
+its keys straight into the pages.  Recurrent mixers keep a fixed-size state per request instead of pages: every request owns a *state row* for its lifetime (``recurrent_state`` hands out per-layer
 tensors ``[max_requests, ...]`` indexed by that row, zeroed when the row is given to a new request), and ``packed``
 describes the step's sequence boundaries and rows to the scan kernels.  Chunked prefill, continuous batching and
 preemption-by-recompute therefore work unchanged for hybrid models.
@@ -198,13 +199,31 @@ class DynamicInferenceContext:
     def last_token_index(self) -> Dict[str, int]:
         return {rid: qs + n - 1 for rid, qs, n, _ in self._plan}
 
+    # -- pages that a layer's own kernel fills ----------------------------------------
+    @property
+    def write_slots(self) -> torch.Tensor:
+        """Cache slot of every token of this step (int64 ``[T]``)."""
+        return self._write_slots
+
+    def kv_pages(self, layer: int, k_shape, v_shape, dtype) -> tuple:
+        """The key and value pages ``[slots, *k_shape]`` / ``[slots, *v_shape]`` of ``layer`` (zeros when first asked for): a layer
+        whose kernel produces keys and values writes them at ``write_slots`` itself."""
+        if layer not in self.kv:
+            n_slots = self.num_blocks * self.block_size
+            self.kv[layer] = (torch.zeros(n_slots, *k_shape, dtype=dtype, device=self._device),
+                              torch.zeros(n_slots, *v_shape, dtype=dtype, device=self._device))
+        return self.kv[layer]
+
+    def latent_pages(self, layer: int, width: int, dtype) -> torch.Tensor:
+        """The latent pages ``[slots, width]`` of ``layer``, as ``kv_pages``."""
+        if layer not in self.latents:
+            self.latents[layer] = torch.zeros(self.num_blocks * self.block_size, width, dtype=dtype, device=self._device)
+        return self.latents[layer]
+
     # -- latent attention over the paged cache ----------------------------------------
     def write_latents(self, layer: int, c_new: torch.Tensor) -> None:
         """Store this step's latents ``[T, r]`` of ``layer`` in their pages."""
-        if layer not in self.latents:
-            self.latents[layer] = torch.zeros(self.num_blocks * self.block_size, c_new.shape[-1], dtype=c_new.dtype,
-                                              device=c_new.device)
-        self.latents[layer][self._write_slots] = c_new
+        self.latent_pages(layer, c_new.shape[-1], c_new.dtype)[self._write_slots] = c_new
 
     def step_latents(self, layer: int) -> torch.Tensor:
         """The latents ``[T, r]`` that ``layer`` wrote for this step's tokens (for a layer that shares them)."""
@@ -212,11 +231,13 @@ class DynamicInferenceContext:
             raise RuntimeError(f"layer {layer} has written no latents for this step")
         return self.latents[layer][self._write_slots]
 
-    def attend_latent(self, layer: int, q_lat: torch.Tensor, c_new: Optional[torch.Tensor], scale: float) -> torch.Tensor:
+    def attend_latent(self, layer: int, q_lat: torch.Tensor, c_new: Optional[torch.Tensor], scale: float,
+                      q_rot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``q_lat [T, H, r]`` (queries carried into the latent space) against the latent pages of ``layer``.  ``c_new
         [T, r]`` are this step's latents, written into their pages first; a layer that shares another layer's latents
-        passes ``None`` and names that layer (whose pages this step already holds).  Returns the softmax-weighted sum of
-        latents, fp32 ``[T, H, r]``."""
+        passes ``None`` and names that layer (whose pages this step already holds), and so does a layer that has written
+        ``latent_pages`` itself.  ``q_rot [T, H, n]`` scores against ``n`` further columns of the page rows, ``gate [T, H]``
+        (pre-activation) scales each head's result.  Returns the softmax-weighted sum of latents, fp32 ``[T, H, r]``."""
         from ..ops import seqmix
 
         if c_new is not None:
@@ -225,7 +246,7 @@ class DynamicInferenceContext:
             raise RuntimeError(f"layer {layer} has written no latents for this step")
         self.kernel_calls += 1
         return seqmix.latent_attention_paged(q_lat, self.latents[layer], self._block_table, self._tok_req, self._tok_len,
-                                             self.block_size, scale, self._max_len)
+                                             self.block_size, scale, self._max_len, q_rot, gate)
 
     def attend_mixed(self, layer: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float,
                      talk: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -264,6 +285,17 @@ class DynamicInferenceContext:
         self.kernel_calls += 1
         return seqmix.window_attention_paged(q, kc, vc, self._block_table, self._tok_req, self._tok_len, self.block_size, scale,
                                              window, slopes, sink, gate, out_scale, self._max_len, dist_bias)
+
+    def attend_sigmoid(self, layer: int, q: torch.Tensor, scale: float, softcap: float = 0.0, head_bias: Optional[torch.Tensor] = None,
+                       turns_back: Optional[torch.Tensor] = None, interleaved: bool = False) -> torch.Tensor:
+        """Grouped-query attention with logistic weights over the pages of cache ``layer``, which the layer has filled through
+        ``kv_pages`` at ``write_slots``: ``q [T, H, d]`` -> ``[T, H * dv]`` (``ops.seqmix.sigmoid_attention_paged``)."""
+        from ..ops import seqmix
+
+        kc, vc = self.kv[layer]
+        self.kernel_calls += 1
+        return seqmix.sigmoid_attention_paged(q, kc, vc, self._block_table, self._tok_req, self._tok_len, self.block_size, scale, softcap,
+                                              head_bias, turns_back, interleaved, self._max_len)
 
     # -- attention over the paged cache --------------------------------------------
     def attend(self, layer: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float) -> torch.Tensor:

@@ -104,10 +104,13 @@ def sort_chunks_by_idxs(x, split_sizes, sorted_idxs):
 
 def group_limited_topk(scores, topk, num_tokens, num_experts, num_groups, group_topk, group_score="topk_sum"):
     """Only experts of the ``group_topk`` best groups compete.  A group ranks by the sum of its best
-    ``topk // group_topk`` scores (``"topk_sum"``) or by its single best score (``"max"``)."""
+    ``topk // group_topk`` scores (``"topk_sum"``), by the sum of its two best (``"top2_sum"``) or by its single best score
+    (``"max"``)."""
     per_group = scores.view(num_tokens, num_groups, -1)
     if group_score == "max":
         group_scores = per_group.amax(dim=-1)
+    elif group_score == "top2_sum":
+        group_scores = per_group.topk(min(2, per_group.shape[-1]), dim=-1)[0].sum(dim=-1)
     else:
         group_scores = per_group.topk(max(1, topk // group_topk), dim=-1)[0].sum(dim=-1)
     group_idx = torch.topk(group_scores, k=group_topk, dim=-1, sorted=False)[1]
@@ -144,7 +147,7 @@ def topk_softmax_with_capacity(logits, topk, capacity_factor=None, pad_to_capaci
             sc = torch.gather(scores, 1, top_idx)
         else:
             sc, top_idx = _topk(scores)
-        probs = sc / (sc.sum(dim=-1, keepdim=True) + 1e-20) if topk > 1 else sc
+        probs = sc / (sc.sum(dim=-1, keepdim=True) + 1e-20) if (topk > 1 or renormalize) else sc
     else:
         raise ValueError(f"invalid score_function {score_function}")
     if scaling_factor:

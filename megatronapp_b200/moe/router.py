@@ -92,15 +92,20 @@ class TopKRouter(MegatronModule):
         fused_ok = (logits.is_cuda and self.score_function == "softmax" and cfg.moe_expert_capacity_factor is None
                     and not cfg.moe_router_group_topk and self.expert_bias is None and self.num_experts <= 256
                     and self.topk <= 8 and logits.dtype in (torch.float32, torch.bfloat16, torch.float16))
-        grouped_ok = (self.score_function == "softmax" and cfg.moe_router_pre_softmax and cfg.moe_router_group_topk
-                      and cfg.moe_router_group_score == "max" and cfg.moe_expert_capacity_factor is None
-                      and self.expert_bias is None and not cfg.moe_router_topk_scaling_factor and not self.training)
-        if grouped_ok:
-            # one warp per token: softmax, groups ranked by their best expert, top-k inside the kept groups
+        # inference: one warp per token -- scores, groups ranked by their best expert(s), top-k inside the kept groups
+        plain = cfg.moe_expert_capacity_factor is None and not self.training
+        grouped_ok = (plain and self.score_function == "softmax" and cfg.moe_router_pre_softmax and cfg.moe_router_group_topk
+                      and cfg.moe_router_group_score == "max" and self.expert_bias is None and not cfg.moe_router_topk_scaling_factor)
+        logistic_ok = (plain and self.score_function == "sigmoid" and (self.topk > 1 or cfg.moe_router_renormalize) and self.topk <= 32
+                       and (not cfg.moe_router_group_topk or cfg.moe_router_group_score in ("max", "top2_sum")))
+        if grouped_ok or logistic_ok:
             from ..ops.seqmix import group_limited_router
 
-            probs, rmap = group_limited_router(logits.float(), self.topk, cfg.moe_router_num_groups,
-                                               cfg.moe_router_group_topk, bool(cfg.moe_router_renormalize))
+            grouped = bool(cfg.moe_router_group_topk)
+            probs, rmap = group_limited_router(
+                logits.float(), self.topk, cfg.moe_router_num_groups if grouped else 1, cfg.moe_router_group_topk if grouped else 1,
+                bool(cfg.moe_router_renormalize) or logistic_ok, self.score_function, self.expert_bias if logistic_ok else None,
+                "top2" if (grouped and cfg.moe_router_group_score == "top2_sum") else "max", float(cfg.moe_router_topk_scaling_factor or 1.0))
             tpe = None
         elif fused_ok:
             # one warp per token: softmax + top-k (+ renormalisation / scaling), dense probs + routing map out

@@ -286,7 +286,8 @@ def mlstm_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_i: torch.T
 # ---------------------------------------------------------------------------
 
 def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, tok_req: torch.Tensor,
-                           tok_len: torch.Tensor, block_size: int, scale: float, max_len: int = 0) -> torch.Tensor:
+                           tok_len: torch.Tensor, block_size: int, scale: float, max_len: int = 0,
+                           q_rot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of every packed query token over the latents of its own sequence, in the latent space.
 
     ``q_lat [T, H, r]``: the query of head ``h`` already carried into the latent space (``W_uk,h^T q_h``), so that
@@ -294,15 +295,24 @@ def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table
     ``block_table [R, max_blocks]``; ``tok_req [T]`` the sequence of each query token, ``tok_len [T]`` how many cached
     tokens it sees (its own included).  Returns ``sum_j softmax_j(score) c_j`` as fp32 ``[T, H, r]``; the caller applies
     the per-head value up-projection.  Scores, softmax and the weighted sum are fp32.  ``max_len`` (the longest visible
-    context, known to the host) lets the kernel split long contexts over several CTAs when the batch has few tokens."""
+    context, known to the host) lets the kernel split long contexts over several CTAs when the batch has few tokens.
+
+    ``q_rot [T, H, n]``: a second query part against ``n`` further columns of the cache rows (``cache [num_slots, r + n]``, one
+    key part shared by all heads): ``score = (q_lat . c + q_rot . k) * scale``; the weighted sum stays over the first ``r``
+    columns.  ``gate [T, H]`` (pre-activation) multiplies head ``h``'s result by its sigmoid."""
     T, H, r = q_lat.shape
+    n_rot = 0 if q_rot is None else q_rot.shape[2]
+    if cache.shape[1] != r + n_rot:
+        raise ValueError(f"latent attention: cache rows of {cache.shape[1]} for queries of {r} + {n_rot}")
     if q_lat.is_cuda:
         kernel_calls["latent_attention_paged"] += 1
         o = torch.empty(T, H, r, dtype=torch.float32, device=q_lat.device)
-        ext().latent_attention_paged(q_lat.contiguous(), cache, block_table, tok_req, tok_len, o, int(block_size),
+        ext().latent_attention_paged(q_lat.contiguous(), None if q_rot is None else q_rot.contiguous(), cache, block_table, tok_req, tok_len,
+                                     None if gate is None else (gate if gate.stride(1) == 1 else gate.contiguous()), o, int(block_size),
                                      float(scale), int(max_len))
         return o
     o = torch.empty(T, H, r, dtype=torch.float32)
+    q = q_lat.float() if q_rot is None else torch.cat([q_lat.float(), q_rot.float()], dim=-1)
     req, lens = tok_req.tolist(), tok_len.tolist()
     t = 0
     while t < T:                                   # tokens of one sequence are contiguous and see growing prefixes
@@ -312,39 +322,51 @@ def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table
         L = lens[e]
         pos = torch.arange(L)
         slots = block_table[req[t]].long()[pos // block_size] * block_size + pos % block_size
-        c = cache[slots].float()                                                        # [L, r]
-        s = torch.einsum("thr,lr->thl", q_lat[t:e + 1].float(), c) * scale
+        c = cache[slots].float()                                                        # [L, r + n]
+        s = torch.einsum("thr,lr->thl", q[t:e + 1], c) * scale
         vis = pos.view(1, 1, L) < torch.tensor(lens[t:e + 1]).view(-1, 1, 1)
-        o[t:e + 1] = torch.einsum("thl,lr->thr", torch.softmax(s.masked_fill(~vis, float("-inf")), -1), c)
+        o[t:e + 1] = torch.einsum("thl,lr->thr", torch.softmax(s.masked_fill(~vis, float("-inf")), -1), c[:, :r])
         t = e + 1
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float()).unsqueeze(-1)
     return o
 
 
 # ---------------------------------------------------------------------------
-# router: softmax scores, groups ranked by their best expert, top-k inside the kept groups
+# router: softmax or logistic scores, groups ranked by their best expert(s), top-k inside the kept groups
 # ---------------------------------------------------------------------------
 
-def group_limited_router(logits: torch.Tensor, topk: int, num_groups: int, keep_groups: int,
-                         renormalize: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
-    """fp32 ``logits [T, E]`` -> dense ``(probs [T, E] fp32, routing_map [T, E] bool)``: softmax over all experts, a
-    group of neighbouring experts scores as its best member, only experts of the ``keep_groups`` best groups compete
-    for the ``topk`` places; chosen scores are divided by their sum (+ 1e-20) when ``renormalize``."""
+def group_limited_router(logits: torch.Tensor, topk: int, num_groups: int, keep_groups: int, renormalize: bool = True,
+                         score_function: str = "softmax", correction: Optional[torch.Tensor] = None, group_score: str = "max",
+                         scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """fp32 ``logits [T, E]`` -> dense ``(probs [T, E] fp32, routing_map [T, E] bool)``: scores are the softmax over all
+    experts or, with ``score_function = "sigmoid"``, the logistic function of each logit; *choice scores* are the scores plus
+    ``correction [E]`` (optional).  A group of neighbouring experts ranks by its best choice score (``group_score = "max"``) or
+    by the sum of its two best (``"top2"``); only experts of the ``keep_groups`` best groups compete for the ``topk`` places,
+    by their choice scores.  The weights are the chosen experts' scores (without the correction), divided by their sum
+    (+ 1e-20) when ``renormalize``, times ``scale``."""
+    if score_function not in ("softmax", "sigmoid") or group_score not in ("max", "top2"):
+        raise ValueError(f"unknown router rule {score_function!r} / {group_score!r}")
     T, E = logits.shape
     if logits.is_cuda:
         kernel_calls["group_limited_router"] += 1
-        probs = torch.zeros(T, E, dtype=torch.float32, device=logits.device)
-        rmap = torch.zeros(T, E, dtype=torch.bool, device=logits.device)
-        ext().group_limited_router(logits.float().contiguous(), probs, rmap, int(topk), int(num_groups), int(keep_groups),
-                                   bool(renormalize))
+        probs = torch.empty(T, E, dtype=torch.float32, device=logits.device)
+        rmap = torch.empty(T, E, dtype=torch.bool, device=logits.device)
+        ext().group_limited_router(logits.float().contiguous(), None if correction is None else correction.float().contiguous(), probs, rmap,
+                                   int(topk), int(num_groups), int(keep_groups), bool(renormalize), score_function == "sigmoid",
+                                   group_score == "top2", float(scale))
         return probs, rmap
-    s = torch.softmax(logits.float(), dim=-1)
-    best = s.view(T, num_groups, E // num_groups).amax(-1)
-    kept = torch.zeros(T, num_groups, dtype=torch.bool).scatter_(1, torch.topk(best, keep_groups, dim=-1).indices, True)
-    masked = s.masked_fill(~kept.repeat_interleave(E // num_groups, dim=1), -1.0)
+    s = torch.softmax(logits.float(), dim=-1) if score_function == "softmax" else torch.sigmoid(logits.float())
+    choice = s if correction is None else s + correction.float()
+    per = choice.view(T, num_groups, E // num_groups)
+    mark = per.amax(-1) if group_score == "max" else per.topk(min(2, E // num_groups), dim=-1).values.sum(-1)
+    kept = torch.zeros(T, num_groups, dtype=torch.bool).scatter_(1, torch.topk(mark, keep_groups, dim=-1).indices, True)
+    masked = choice.masked_fill(~kept.repeat_interleave(E // num_groups, dim=1), float("-inf"))
     idx = torch.topk(masked, topk, dim=-1).indices
     w = torch.gather(s, 1, idx)
     if renormalize:
         w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    w = w * scale
     return torch.zeros_like(s).scatter_(1, idx, w), torch.zeros(T, E, dtype=torch.bool).scatter_(1, idx, True)
 
 
@@ -815,3 +837,243 @@ def gelu_mul(g: torch.Tensor, e: torch.Tensor) -> torch.Tensor:
         ext().gelu_mul(g if g.stride(1) == 1 else g.contiguous(), e if e.stride(1) == 1 else e.contiguous(), y)
         return y
     return (F.gelu(g.float(), approximate="tanh") * e.float()).to(g.dtype)
+
+
+# ---------------------------------------------------------------------------
+# gated additions of two sublayers, fused with the norm(s) of what follows
+# ---------------------------------------------------------------------------
+
+def gated_add_norm(x: torch.Tensor, a: Optional[torch.Tensor], gate_a: Optional[torch.Tensor], bias_a: Optional[torch.Tensor],
+                   b: Optional[torch.Tensor], gate_b: Optional[torch.Tensor], bias_b: Optional[torch.Tensor], weight1: torch.Tensor,
+                   weight2: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype, center: bool = True):
+    """``x`` fp32 ``[T, W]`` is updated in place by ``+ sigmoid(gate_a + bias_a) * a + sigmoid(gate_b + bias_b) * b`` (each
+    addend optional, a missing gate is one), then normed once for two readers: ``n = layer_norm(x)`` (RMS norm unless ``center``,
+    no bias), ``h1 = n * weight1``, ``h2 = n * weight2``.  Gates, sums and statistics are fp32; ``h1`` and ``h2`` leave in
+    ``out_dtype``.  Returns ``(x, h1, h2 or None)``."""
+    if x.is_cuda:
+        kernel_calls["gated_add_norm"] += 1
+        h1 = torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        h2 = torch.empty(x.shape, dtype=out_dtype, device=x.device) if weight2 is not None else None
+        fix = lambda t: t if (t is None or t.stride(1) == 1) else t.contiguous()  # noqa: E731
+        ext().gated_add_norm(x, fix(a), fix(gate_a), bias_a, fix(b), fix(gate_b), bias_b, weight1, weight2, h1, h2, float(eps), bool(center))
+        return x, h1, h2
+    for t, g, c in ((a, gate_a, bias_a), (b, gate_b, bias_b)):
+        if t is None:
+            continue
+        f = 1.0
+        if g is not None:
+            f = torch.sigmoid(g.float() + (c.float() if c is not None else 0.0))
+        x.add_(f * t.float())
+    n = x - x.mean(-1, keepdim=True) if center else x
+    n = n * torch.rsqrt(n.pow(2).mean(-1, keepdim=True) + eps)
+    return x, (n * weight1.float()).to(out_dtype), None if weight2 is None else (n * weight2.float()).to(out_dtype)
+
+
+# ---------------------------------------------------------------------------
+# rotary positions of whole heads, with an optional norm, written where the consumer reads
+# ---------------------------------------------------------------------------
+
+def rotary_turns(rot_dims: int, base: float, scaling: Optional[dict] = None, device=None) -> Tuple[Optional[torch.Tensor], float]:
+    """``(turns [n, 2], amplitude)`` of a rotary position over ``rot_dims`` dimensions: pair ``i`` turns by ``base^(-2 i /
+    rot_dims)`` radians per position.  The rates are kept in full turns as a sum of two fp32 numbers, so that the angle of a far
+    position (``position * turns`` modulo one) keeps fp32 accuracy.  ``scaling`` (``factor``, ``original``, ``fast``, ``slow``):
+    YaRN (Peng et al., "YaRN: Efficient Context Window Extension of Large Language Models"): pairs that make fewer than ``slow``
+    turns over the original length turn ``factor`` times slower, those above ``fast`` turns keep their rate, a ramp between;
+    cosine and sine are multiplied by ``0.1 ln(factor) + 1``."""
+    import math
+
+    n = rot_dims // 2
+    if n <= 0:
+        return None, 1.0
+    i = torch.arange(n, dtype=torch.float64)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / rot_dims)
+    amp = 1.0
+    if scaling:
+        factor, original = float(scaling["factor"]), float(scaling["original"])
+        edge = lambda turns: rot_dims * math.log(original / (2.0 * math.pi * float(turns))) / (2.0 * math.log(float(base)))  # noqa: E731
+        lo = max(math.floor(edge(scaling["fast"])), 0)
+        hi = min(math.ceil(edge(scaling["slow"])), rot_dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        f = f / factor * ramp + f * (1.0 - ramp)
+        amp = 0.1 * math.log(factor) + 1.0
+    t = f / (2.0 * math.pi)
+    high = t.float()
+    return torch.stack([high, (t - high.double()).float()], dim=1).contiguous().to(device), amp
+
+
+def _turn_tables(turns: torch.Tensor, positions: torch.Tensor, amplitude: float) -> Tuple[torch.Tensor, torch.Tensor]:
+    ang = positions.double().unsqueeze(-1) * turns.double().sum(-1)
+    ang = (ang - ang.round()) * 6.283185307179586
+    return (torch.cos(ang) * amplitude).float(), (torch.sin(ang) * amplitude).float()
+
+
+class HeadPart:
+    """One operand of ``head_rotary``: the heads ``x [T, H, d]`` (unit inner stride, any head and row stride), how they are
+    treated, and where the result goes.
+
+    ``turns [n, 2]`` (``rotary_turns``; ``None``: nothing turns), pairs ``(i, i + n)`` or ``interleaved`` ``(2 i, 2 i + 1)``,
+    ``amplitude`` on cosine and sine, ``back`` for the negative angle; ``rms``: every head is divided by its root mean square
+    after the rotation, times ``weight [d]`` if given.  ``out``: ``[T, H, d']`` with ``d' >= d`` (the columns from ``d`` on
+    become zero), row ``t`` at ``out[t]``; ``pages``: ``[slots, H, d]``, row ``t`` at ``pages[slots[t]]``; either may be absent."""
+
+    def __init__(self, x, turns=None, interleaved=False, amplitude=1.0, back=False, rms=False, weight=None, out=None, pages=None):
+        self.x, self.turns, self.interleaved, self.amplitude, self.back = x, turns, bool(interleaved), float(amplitude), bool(back)
+        self.rms, self.weight, self.out, self.pages = bool(rms), weight, out, pages
+
+
+def head_rotary(parts: Sequence[HeadPart], positions: torch.Tensor, eps: float, slots: Optional[torch.Tensor] = None) -> None:
+    """Rotate / norm up to three groups of heads in one launch (queries, keys and values of a token, say) and write them to
+    their outputs and cache pages.  ``positions [T]``, ``slots [T]`` int64.  Angles and statistics are fp32."""
+    if not 1 <= len(parts) <= 3:
+        raise ValueError("head_rotary takes one to three parts")
+    if positions.is_cuda:
+        kernel_calls["head_rotary"] += 1
+        ext().head_rotary([p.x for p in parts], [p.turns for p in parts], [p.weight for p in parts], [p.out for p in parts],
+                          [p.pages for p in parts], [p.interleaved for p in parts], [p.amplitude for p in parts],
+                          [p.back for p in parts], [p.rms for p in parts], positions, slots, float(eps))
+        return
+    for p in parts:
+        y = p.x.float().clone()
+        if p.turns is not None:
+            n = p.turns.shape[0]
+            cs, sn = _turn_tables(p.turns, positions, p.amplitude)
+            cs, sn = cs.unsqueeze(1), (-sn if p.back else sn).unsqueeze(1)
+            a, b = (slice(0, 2 * n, 2), slice(1, 2 * n, 2)) if p.interleaved else (slice(0, n), slice(n, 2 * n))
+            u, w = y[..., a].clone(), y[..., b].clone()
+            y[..., a] = u * cs - w * sn
+            y[..., b] = w * cs + u * sn
+        if p.rms:
+            y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+            if p.weight is not None:
+                y = y * p.weight.float()
+        d = y.shape[-1]
+        if p.out is not None:
+            p.out[..., :d] = y.to(p.out.dtype)
+            p.out[..., d:] = 0
+        if p.pages is not None:
+            p.pages[slots] = y.to(p.pages.dtype)
+
+
+def latent_head_assemble(q: torch.Tensor, k: torch.Tensor, k_rot: torch.Tensor, v: torch.Tensor, turns: Optional[torch.Tensor],
+                         interleaved: bool, amplitude: float, positions: torch.Tensor, q_out: torch.Tensor, k_out: torch.Tensor,
+                         v_out: torch.Tensor) -> None:
+    """Whole heads of a rotary latent attention, padded with zeros to the outputs' width: ``q_out = [q_n | R q_r | 0]`` from ``q
+    [T, H, d + n]`` (its last ``n`` dimensions turn), ``k_out = [k | k_rot | 0]`` with ``k_rot [T, n]`` (already turned) repeated
+    over the heads, ``v_out = [v | 0]``."""
+    T, H, d = k.shape
+    n = k_rot.shape[1]
+    if q.is_cuda:
+        kernel_calls["latent_head_assemble"] += 1
+        ext().latent_head_assemble(q.contiguous(), k.contiguous(), k_rot if k_rot.stride(1) == 1 else k_rot.contiguous(), v.contiguous(), turns,
+                                   bool(interleaved), float(amplitude), positions, q_out, k_out, v_out)
+        return
+    q_out.zero_(), k_out.zero_(), v_out.zero_()
+    q_out[..., :d] = q[..., :d]
+    head_rotary([HeadPart(q[..., d:], turns, interleaved, amplitude, out=q_out[..., d:d + n])], positions, 0.0)
+    k_out[..., :d], k_out[..., d:d + n], v_out[..., :v.shape[2]] = k, k_rot.unsqueeze(1), v
+
+
+def head_gate(o: torch.Tensor, gate: Optional[torch.Tensor], out_dtype: torch.dtype) -> torch.Tensor:
+    """``o [T, H, dv]`` (unit inner stride): head ``h`` times ``sigmoid(gate[:, h])`` (``gate [T, H]`` pre-activation, any row
+    stride; ``None``: as it is) -> contiguous ``[T, H, dv]`` in ``out_dtype``."""
+    if gate is None:
+        return o.to(out_dtype).contiguous()
+    if o.is_cuda:
+        kernel_calls["head_gate"] += 1
+        y = torch.empty(o.shape, dtype=out_dtype, device=o.device)
+        ext().head_gate(o if o.stride(2) == 1 else o.contiguous(), gate if gate.stride(1) == 1 else gate.contiguous(), y)
+        return y
+    return (o.float() * torch.sigmoid(gate.float()).unsqueeze(-1)).to(out_dtype).contiguous()
+
+
+# ---------------------------------------------------------------------------
+# paged grouped-query attention whose weights are logistic functions of the scores
+# ---------------------------------------------------------------------------
+
+def sigmoid_attention_paged(q: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor, block_table: torch.Tensor,
+                            tok_req: torch.Tensor, tok_len: torch.Tensor, block_size: int, scale: float, softcap: float = 0.0,
+                            head_bias: Optional[torch.Tensor] = None, turns_back: Optional[torch.Tensor] = None,
+                            interleaved: bool = False, max_len: int = 0) -> torch.Tensor:
+    """``q [T, H, d]`` against paged keys ``[slots, G, d]`` and values ``[slots, G, dv]``; the token at position
+    ``i = tok_len[t] - 1`` sees the keys ``j <= i`` of its own sequence::
+
+        s_j = cap(q . k_j * scale) + head_bias[h],  cap(z) = softcap tanh(z / softcap) (softcap 0: z);   o = sum_j sigmoid(s_j) v_j
+
+    The weights are not normalised.  ``turns_back [n, 2]`` (``rotary_turns``): the pairs of the result are turned by minus the
+    token's own angle, in the layout given by ``interleaved``: values that were rotated by their positions before they were
+    cached then enter by their distance.  Scores, weights, sums and angles are fp32.  Returns ``[T, H * dv]`` in ``q``'s dtype."""
+    T, H, d = q.shape
+    G, dv = kcache.shape[1], vcache.shape[2]
+    if q.is_cuda:
+        kernel_calls["sigmoid_attention_paged"] += 1
+        o = torch.empty(T, H * dv, dtype=q.dtype, device=q.device)
+        ext().sigmoid_attention_paged(_rows3(q), kcache, vcache, block_table, tok_req, tok_len,
+                                      None if head_bias is None else head_bias.float().contiguous(), turns_back, o, int(block_size),
+                                      float(scale), float(softcap), bool(interleaved), int(max_len))
+        return o
+    o = torch.empty(T, H, dv, dtype=torch.float32)
+    req, lens = tok_req.tolist(), tok_len.tolist()
+    rep = H // G
+    t = 0
+    while t < T:
+        e = t
+        while e + 1 < T and req[e + 1] == req[t]:
+            e += 1
+        L = max(lens[t:e + 1])
+        pos = torch.arange(L)
+        slots = block_table[req[t]].long()[pos // block_size] * block_size + pos % block_size
+        kk = kcache[slots].float().repeat_interleave(rep, dim=1)
+        vv = vcache[slots].float().repeat_interleave(rep, dim=1)
+        s = torch.einsum("thd,lhd->htl", q[t:e + 1].float(), kk) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
+        if head_bias is not None:
+            s = s + head_bias.float().view(H, 1, 1)
+        vis = pos.view(1, 1, L) < torch.tensor(lens[t:e + 1]).view(1, -1, 1)
+        o[t:e + 1] = torch.einsum("htl,lhv->thv", torch.sigmoid(s).masked_fill(~vis, 0.0), vv)
+        t = e + 1
+    if turns_back is not None:
+        out = torch.empty(T, H, dv, dtype=torch.float32)
+        head_rotary([HeadPart(o, turns_back, interleaved, back=True, out=out)], tok_len.long() - 1, 0.0)
+        o = out
+    return o.reshape(T, H * dv).to(q.dtype)
+
+
+# ---------------------------------------------------------------------------
+# real-gated linear recurrent unit with block-diagonal gates
+# ---------------------------------------------------------------------------
+
+def rglru_scan(u: torch.Tensor, w_gates: torch.Tensor, b_gates: torch.Tensor, lam: torch.Tensor, y_pre: Optional[torch.Tensor],
+               pb: PackedBatch, state: torch.Tensor, decay_scale: float = 8.0) -> torch.Tensor:
+    """``u [T, C]``, ``w_gates [B, 2, n, n]`` and ``b_gates [B, 2, n]`` (``B n = C``; index 0 the recurrence gate, 1 the input
+    gate, each ``[out, in]``), ``lam [C]``, ``state [rows, C]`` fp32 -> ``[T, C]`` in ``u``'s dtype.  Per part ``b`` of the channels::
+
+        r, i = sigmoid(w_gates[b, 0] u_b + b_gates[b, 0]), sigmoid(w_gates[b, 1] u_b + b_gates[b, 1])
+        log_a = -decay_scale * r * softplus(lam);   S <- exp(log_a) S + sqrt(1 - exp(2 log_a)) i u;   y = S * gelu_tanh(y_pre)
+
+    The gates' sums, decays and the state are fp32 (Griffin's recurrent block: De et al., "Griffin: Mixing Gated Linear
+    Recurrences with Local Attention for Efficient Language Models")."""
+    T, C = u.shape
+    B, n = w_gates.shape[0], w_gates.shape[2]
+    if u.is_cuda:
+        kernel_calls["rglru_scan"] += 1
+        y = torch.empty(T, C, dtype=u.dtype, device=u.device)
+        fix = lambda t: t if (t is None or t.stride(1) == 1) else t.contiguous()  # noqa: E731
+        ext().rglru_scan(fix(u), w_gates, b_gates, lam, fix(y_pre), pb.cu, pb.slots, state, y, float(decay_scale), pb.max_len)
+        return y
+    uf = u.float()
+    pre = torch.einsum("tbi,bgoi->tgbo", uf.view(T, B, n), w_gates.float()) + b_gates.float().transpose(0, 1)
+    r, i = torch.sigmoid(pre[:, 0]).reshape(T, C), torch.sigmoid(pre[:, 1]).reshape(T, C)
+    log_a = -decay_scale * r * F.softplus(lam.float(), threshold=30.0)
+    a, put = torch.exp(log_a), torch.sqrt(-torch.expm1(2.0 * log_a)) * i * uf
+    out = torch.empty(T, C, dtype=torch.float32)
+    for k in range(pb.num_seqs):
+        lo, hi, row = pb.cu_host[k], pb.cu_host[k + 1], pb.slots_host[k]
+        S = state[row].clone()
+        for t in range(lo, hi):
+            S = a[t] * S + put[t]
+            out[t] = S
+        state[row] = S
+    if y_pre is not None:
+        out = out * F.gelu(y_pre.float(), approximate="tanh")
+    return out.to(u.dtype)

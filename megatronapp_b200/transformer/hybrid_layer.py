@@ -1,7 +1,8 @@
 """Layers over an fp32 residual stream with an arbitrary sequence mixer, and the blocks that stack them: pre-norm
 (``ResidualF32Layer`` / ``ResidualF32Block``), norm on the sublayer's output (``OutputNormF32Layer`` /
-``OutputNormF32Block``), several streams (``StreamLayer`` / ``StreamBlock``) and one norm read by mixer and feed-forward side
-by side (``ParallelF32Layer`` / ``ParallelF32Block``), further down.
+``OutputNormF32Block``), several streams (``StreamLayer`` / ``StreamBlock``), one norm read by mixer and feed-forward side
+by side (``ParallelF32Layer`` / ``ParallelF32Block``), and side by side with a norm and a gate each (``DualNormF32Layer`` /
+``DualNormF32Block``), further down.
 
 ``x <- x + mixer(norm1(x));  x <- x + mlp(norm2(x))`` (the second half is absent for a layer without feed-forward).
 The stream ``x`` stays fp32 whatever the parameter dtype; every addition is fused into the norm that follows it
@@ -343,3 +344,100 @@ class ParallelF32Block(MegatronModule):
             if self.tap is not None:
                 self.tap(k, x)
         return x if self.final_layernorm is None else h
+
+
+class SublayerSum:
+    """Outputs of a layer's sublayers waiting to be added to the stream: ``sigmoid(gate + bias) * out`` each (no gate: ``out``)."""
+
+    def __init__(self):
+        self.terms = []
+
+    def add(self, out, gate=None, bias=None):
+        self.terms.append((out, gate, bias))
+
+    def operands(self, W):
+        """``(a, gate_a, bias_a, b, gate_b, bias_b)`` as packed ``[T, W]`` rows for ``ops.seqmix.gated_add_norm``."""
+        flat = []
+        for out, gate, bias in self.terms:
+            flat += [out.reshape(-1, W), None if gate is None else gate.reshape(-1, W), bias]
+        return flat + [None] * (6 - len(flat))
+
+
+class DualNormF32Layer(MegatronModule):
+    """Mixer and feed-forward side by side, each behind a norm of its own and with a gate on its output::
+
+        a = norm(x) * w1;  b = norm(x) * w2;   x <- x + sigmoid(R1 a + r1) * mixer(a) + sigmoid(R2 b + r2) * mlp(b)
+
+    Both norms read the same ``x``, so its statistics are computed once; ``norm`` is a layer norm without bias (``center``) or an
+    RMS norm.  ``gated = False`` leaves the gates out.  The stream is fp32; the additions, the gates' activations and the next
+    layer's two norms are one kernel (``ops.seqmix.gated_add_norm``), so a layer takes ``(h1, h2)`` and returns a ``SublayerSum``."""
+
+    def __init__(self, config, layer_number: int, mixer: nn.Module, mlp: Optional[nn.Module] = None, gated: bool = True):
+        super().__init__(config)
+        from ..parallel.tp_layers import ColumnParallelLinear
+
+        self.layer_number = layer_number
+        W, eps = config.hidden_size, config.layernorm_epsilon
+        self.mixer, self.mlp = mixer, mlp
+        col = dict(config=config, init_method=config.init_method, bias=True, skip_bias_add=True, gather_output=True)
+        self.input_norm_weight = ResidualRMSNorm(config, W, eps).weight
+        self.mixer_gate = ColumnParallelLinear(W, W, **col) if gated else None
+        self.pre_mlp_norm_weight = ResidualRMSNorm(config, W, eps).weight if mlp is not None else None
+        self.mlp_gate = ColumnParallelLinear(W, W, **col) if (gated and mlp is not None) else None
+        if mlp is not None and hasattr(mlp, "set_layer_number"):
+            mlp.set_layer_number(layer_number)
+
+    def forward(self, h1, h2=None, inference_context=None, cache_index=None) -> SublayerSum:
+        pending = SublayerSum()
+        with _scope("transformer_layer", layer=self.layer_number):
+            out, bias = self.mixer(h1, inference_context=inference_context,
+                                   cache_index=self.layer_number if cache_index is None else cache_index)
+            pending.add(out if bias is None else out + bias, *(self.mixer_gate(h1) if self.mixer_gate is not None else (None, None)))
+            if self.mlp is not None:
+                out, bias = self.mlp(h2)
+                pending.add(out if bias is None else out + bias, *(self.mlp_gate(h2) if self.mlp_gate is not None else (None, None)))
+        return pending
+
+
+class DualNormF32Block(MegatronModule):
+    """A stack of ``DualNormF32Layer`` runs followed by the final norm.  ``layer_builders[i](i)`` builds layer object ``i``; ``runs``
+    lists, depth by depth, which object runs there (default: each once, in order); run ``k`` uses cache / state index ``k``.
+    ``center`` as in the layer.  ``tap(run, residual)`` receives the stream after every run."""
+
+    def __init__(self, config, layer_builders: List[Callable[[int], DualNormF32Layer]], runs: Optional[List[int]] = None,
+                 post_process: bool = True, center: bool = True):
+        super().__init__(config)
+        self.layers = nn.ModuleList([build(i) for i, build in enumerate(layer_builders)])
+        self.runs = list(range(len(self.layers))) if runs is None else [int(r) for r in runs]
+        if any(not 0 <= r < len(self.layers) for r in self.runs):
+            raise ValueError("a run names a layer that does not exist")
+        self.center, self.eps = bool(center), config.layernorm_epsilon
+        self.final_norm_weight = ResidualRMSNorm(config, config.hidden_size, self.eps).weight if post_process else None
+        self.input_tensor = None
+        self.tap = None
+
+    def set_input_tensor(self, t):
+        self.input_tensor = t
+
+    def forward(self, hidden_states, inference_context=None):
+        from ..ops import seqmix
+
+        x = hidden_states if self.input_tensor is None else self.input_tensor
+        if x.dtype != torch.float32:
+            x = x.float()
+        shape, W, dt = x.shape, x.shape[-1], self.config.params_dtype
+        x2 = x.reshape(-1, W)
+        pending, n = SublayerSum(), len(self.runs)
+        for k in range(n + 1):
+            layer = self.layers[self.runs[k]] if k < n else None
+            w1 = layer.input_norm_weight if layer is not None else self.final_norm_weight
+            w2 = layer.pre_mlp_norm_weight if layer is not None else None
+            if w1 is None:                                          # no final norm on this stage: only the last addition
+                w1 = torch.ones(W, dtype=dt, device=x.device)
+            _, h1, h2 = seqmix.gated_add_norm(x2, *pending.operands(W), w1, w2, self.eps, dt, self.center)
+            if self.tap is not None and k > 0:
+                self.tap(k - 1, x2.view(shape))
+            if layer is None:
+                break
+            pending = layer(h1.view(shape), None if h2 is None else h2.view(shape), inference_context=inference_context, cache_index=k)
+        return h1.view(shape) if self.final_norm_weight is not None else x2.view(shape)
