@@ -221,6 +221,22 @@ int attn_fwd(const AttnArgs& a, cudaStream_t s);
 int attn_bwd(const AttnArgs& a, cudaStream_t s);
 const char* attn_last_error();
 
+// causal attention with logistic weights over packed prompts (tcgen05)
+struct SigAttnArgs {
+  const void *q, *k, *v;   // [T, H, d], [T, G, d], [T, G, d] contiguous, padded with zeros to d = 64 or 128
+  void* o;                 // [T, H, dv]
+  const int* cu;           // [n_seqs + 1]
+  const float* bias;       // [H] added to the capped score (nullptr: none)
+  const float* table;      // [T, n_pairs, 2] cosine / sine by which the result's pairs are turned back (nullptr: none)
+  int n_tok, n_seqs, max_len, H, G, d, dv;
+  int n_pairs, interleaved;  // pairs (2 i, 2 i + 1), or (i, n_pairs + i) with the second half of a value at column d / 2
+  float scale, softcap;    // softcap 0: none
+  bool is_bf16;
+};
+int sigmoid_attn_fwd(const SigAttnArgs& a, cudaStream_t s);
+int sigmoid_attn_status();   // 1: a kernel of this process gave up on a wait
+const char* sigmoid_attn_last_error();
+
 // ---------------------------------------------------------------- comm
 void push_flags_barrier(uint32_t* const* peer_flags, int rank, int size, int slot, uint32_t epoch,
                         cudaStream_t s);

@@ -157,55 +157,73 @@ void mlstm_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor&
   count(); check_last_error("mlstm_scan");
 }
 
-void latent_attention_paged(const Tensor& q, const Tensor& cache, const Tensor& block_table, const Tensor& tok_req, const Tensor& tok_len,
-                            Tensor out, int64_t block_size, double scale, int64_t max_len) {
-  const bool bf16 = act_is_bf16(q, "q_lat");
-  TORCH_CHECK(q.dim() == 3 && q.is_contiguous(), "q_lat must be contiguous [T, H, r]");
-  TORCH_CHECK(cache.scalar_type() == q.scalar_type() && cache.dim() == 2 && cache.is_contiguous() && cache.size(1) == q.size(2),
-              "cache must be [slots, r] in q_lat's dtype");
-  check_i32(block_table, "block_table"); check_i32(tok_req, "tok_req"); check_i32(tok_len, "tok_len"); check_f32(out, "out");
-  TORCH_CHECK(block_table.dim() == 2 && tok_req.numel() == q.size(0) && tok_len.numel() == q.size(0) && out.numel() == q.numel(),
-              "bad shapes");
-  b200seq::LatentAttnArgs p{};
-  p.q = q.data_ptr(); p.cache = cache.data_ptr();
-  p.block_table = block_table.data_ptr<int>(); p.tok_req = tok_req.data_ptr<int>(); p.tok_len = tok_len.data_ptr<int>();
-  p.out = out.data_ptr<float>();
-  p.H = static_cast<int>(q.size(1)); p.r = static_cast<int>(q.size(2)); p.block_size = static_cast<int>(block_size);
-  p.max_blocks = static_cast<int>(block_table.size(1)); p.scale = static_cast<float>(scale);
-  c10::cuda::CUDAGuard g(q.device());
-  p.n_splits = b200seq::latent_attention_splits(p.H, p.r, static_cast<int>(q.size(0)), static_cast<int>(max_len));
-  const int64_t vec = 16 / static_cast<int64_t>(cache.element_size());
-  p.vec_ok = (p.r % vec == 0 && reinterpret_cast<uintptr_t>(cache.data_ptr()) % 16 == 0) ? 1 : 0;
-  Tensor ws;
-  if (p.n_splits > 1) {
-    ws = torch::empty({q.size(0), q.size(1), p.n_splits, q.size(2) + 2}, out.options());
-    p.ws = ws.data_ptr<float>();
-  }
-  TORCH_CHECK(b200seq::latent_attention_paged(p, static_cast<int>(q.size(0)), bf16, cur_stream()), "latent_attention_paged: rank ", p.r,
-              " above the largest kernel instance (1024)");
-  count(p.n_splits > 1 ? 2 : 1); check_last_error("latent_attention_paged");
-}
-
-void group_limited_router(const Tensor& logits, Tensor probs, Tensor rmap, int64_t topk, int64_t groups, int64_t keep, bool renorm) {
-  check_f32(logits, "logits"); check_f32(probs, "probs");
-  TORCH_CHECK(logits.dim() == 2 && probs.sizes() == logits.sizes() && rmap.sizes() == logits.sizes() && rmap.scalar_type() == at::kBool &&
-              rmap.is_contiguous(), "bad shapes");
-  c10::cuda::CUDAGuard g(logits.device());
-  TORCH_CHECK(b200seq::group_limited_router(logits.data_ptr<float>(), probs.data_ptr<float>(), rmap.data_ptr<bool>(),
-                                            static_cast<int>(logits.size(0)), static_cast<int>(logits.size(1)), static_cast<int>(topk),
-                                            static_cast<int>(groups), static_cast<int>(keep), renorm, cur_stream()),
-              "group_limited_router: unsupported sizes (experts ", logits.size(1), ", groups ", groups, ", top ", topk, ")");
-  count(); check_last_error("group_limited_router");
-}
-
-
-// ---- side-by-side mixer, minGRU, clamped gated activation ------------------------------------------------------------------
 const void* opt_ptr(const c10::optional<Tensor>& t) { return (t.has_value() && t->defined()) ? t->data_ptr() : nullptr; }
 void check_act2(const Tensor& t, const Tensor& like, const char* name) {   // [T, C], unit inner stride, free row stride
   TORCH_CHECK(t.is_cuda() && t.dim() == 2 && t.stride(1) == 1 && t.scalar_type() == like.scalar_type(), name,
               " must be a [T, C] CUDA tensor with unit inner stride in the activation dtype");
 }
 
+void latent_attention_paged(const Tensor& q, c10::optional<Tensor> q_rot, const Tensor& cache, const Tensor& block_table, const Tensor& tok_req,
+                            const Tensor& tok_len, c10::optional<Tensor> gate, Tensor out, int64_t block_size, double scale, int64_t max_len) {
+  const bool bf16 = act_is_bf16(q, "q_lat");
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous(), "q_lat must be contiguous [T, H, r]");
+  b200seq::LatentAttnArgs p{};
+  if (opt_ptr(q_rot) != nullptr) {
+    TORCH_CHECK(q_rot->scalar_type() == q.scalar_type() && q_rot->dim() == 3 && q_rot->is_contiguous() && q_rot->size(0) == q.size(0) &&
+                q_rot->size(1) == q.size(1), "q_rot must be contiguous [T, H, n] in q_lat's dtype");
+    p.q_rot = q_rot->data_ptr(); p.n_rot = static_cast<int>(q_rot->size(2));
+  }
+  TORCH_CHECK(cache.scalar_type() == q.scalar_type() && cache.dim() == 2 && cache.is_contiguous() && cache.size(1) == q.size(2) + p.n_rot,
+              "cache must be [slots, r (+ n)] in q_lat's dtype");
+  check_i32(block_table, "block_table"); check_i32(tok_req, "tok_req"); check_i32(tok_len, "tok_len"); check_f32(out, "out");
+  TORCH_CHECK(block_table.dim() == 2 && tok_req.numel() == q.size(0) && tok_len.numel() == q.size(0) && out.numel() == q.numel(),
+              "bad shapes");
+  if (opt_ptr(gate) != nullptr) {
+    check_act2(*gate, q, "gate");
+    TORCH_CHECK(gate->size(0) == q.size(0) && gate->size(1) == q.size(1), "gate must be [T, H]");
+    p.gate = gate->data_ptr(); p.ldg = gate->stride(0);
+  }
+  p.q = q.data_ptr(); p.cache = cache.data_ptr();
+  p.block_table = block_table.data_ptr<int>(); p.tok_req = tok_req.data_ptr<int>(); p.tok_len = tok_len.data_ptr<int>();
+  p.out = out.data_ptr<float>();
+  p.H = static_cast<int>(q.size(1)); p.r = static_cast<int>(q.size(2)); p.block_size = static_cast<int>(block_size);
+  p.max_blocks = static_cast<int>(block_table.size(1)); p.scale = static_cast<float>(scale);
+  c10::cuda::CUDAGuard g(q.device());
+  p.n_splits = b200seq::latent_attention_splits(p.H, p.r + p.n_rot, static_cast<int>(q.size(0)), static_cast<int>(max_len));
+  const int64_t vec = 16 / static_cast<int64_t>(cache.element_size());
+  p.vec_ok = ((p.r + p.n_rot) % vec == 0 && reinterpret_cast<uintptr_t>(cache.data_ptr()) % 16 == 0) ? 1 : 0;
+  Tensor ws;
+  if (p.n_splits > 1) {
+    ws = torch::empty({q.size(0), q.size(1), p.n_splits, q.size(2) + 2}, out.options());
+    p.ws = ws.data_ptr<float>();
+  }
+  TORCH_CHECK(b200seq::latent_attention_paged(p, static_cast<int>(q.size(0)), bf16, cur_stream()), "latent_attention_paged: rank ", p.r + p.n_rot,
+              " above the largest kernel instance (1024)");
+  count(p.n_splits > 1 ? 2 : 1); check_last_error("latent_attention_paged");
+}
+
+void group_limited_router(const Tensor& logits, c10::optional<Tensor> correction, Tensor probs, Tensor rmap, int64_t topk, int64_t groups,
+                          int64_t keep, bool renorm, bool sigmoid, bool top2, double scale) {
+  check_f32(logits, "logits"); check_f32(probs, "probs");
+  TORCH_CHECK(logits.dim() == 2 && probs.sizes() == logits.sizes() && rmap.sizes() == logits.sizes() && rmap.scalar_type() == at::kBool &&
+              rmap.is_contiguous(), "bad shapes");
+  const float* cp = nullptr;
+  if (opt_ptr(correction) != nullptr) {
+    check_f32(*correction, "correction");
+    TORCH_CHECK(correction->numel() == logits.size(1), "correction must be [experts]");
+    cp = correction->data_ptr<float>();
+  }
+  c10::cuda::CUDAGuard g(logits.device());
+  TORCH_CHECK(b200seq::group_limited_router(logits.data_ptr<float>(), cp, probs.data_ptr<float>(), rmap.data_ptr<bool>(),
+                                            static_cast<int>(logits.size(0)), static_cast<int>(logits.size(1)), static_cast<int>(topk),
+                                            static_cast<int>(groups), static_cast<int>(keep), renorm, sigmoid, top2, static_cast<float>(scale),
+                                            cur_stream()),
+              "group_limited_router: unsupported sizes (experts ", logits.size(1), ", groups ", groups, ", top ", topk, ")");
+  count(); check_last_error("group_limited_router");
+}
+
+
+// ---- side-by-side mixer, minGRU, clamped gated activation ------------------------------------------------------------------
 void norm_add(Tensor x, const Tensor& a, c10::optional<Tensor> b, c10::optional<Tensor> wa, c10::optional<Tensor> wb,
               c10::optional<Tensor> w, Tensor y, double eps, double w_off, c10::optional<Tensor> extra, c10::optional<Tensor> next_w) {
   check_f32(x, "x");
@@ -574,6 +592,221 @@ void window_attention_paged(const Tensor& q, const Tensor& kcache, const Tensor&
   count(p.n_splits > 1 ? 2 : 1); check_last_error("window_attention_paged");
 }
 
+void sigmoid_attention_paged(const Tensor& q, const Tensor& kcache, const Tensor& vcache, const Tensor& block_table, const Tensor& tok_req,
+                             const Tensor& tok_len, c10::optional<Tensor> head_bias, c10::optional<Tensor> turns_back, Tensor out,
+                             int64_t block_size, double scale, double softcap, bool interleaved, int64_t max_len) {
+  const bool bf16 = act_is_bf16(q, "q");
+  check_rows(q, "q");
+  TORCH_CHECK(kcache.scalar_type() == q.scalar_type() && vcache.scalar_type() == q.scalar_type() && kcache.dim() == 3 && vcache.dim() == 3 &&
+              kcache.is_contiguous() && vcache.is_contiguous() && kcache.size(2) == q.size(2) && vcache.size(1) == kcache.size(1),
+              "caches must be contiguous [slots, G, d] / [slots, G, dv] in q's dtype");
+  check_i32(block_table, "block_table"); check_i32(tok_req, "tok_req"); check_i32(tok_len, "tok_len");
+  b200seq::WindowAttnArgs p{};
+  p.n_tok = static_cast<int>(q.size(0));
+  p.H = static_cast<int>(q.size(1)); p.G = static_cast<int>(kcache.size(1)); p.d = static_cast<int>(q.size(2));
+  p.dv = static_cast<int>(vcache.size(2));
+  TORCH_CHECK(block_table.dim() == 2 && tok_req.numel() == q.size(0) && tok_len.numel() == q.size(0), "bad packed-batch tensors");
+  TORCH_CHECK(out.scalar_type() == q.scalar_type() && out.is_contiguous() && out.numel() == q.size(0) * p.H * p.dv, "bad out");
+  p.q = q.data_ptr(); p.ldq = q.stride(0); p.kcache = kcache.data_ptr(); p.vcache = vcache.data_ptr();
+  p.block_table = block_table.data_ptr<int>(); p.tok_req = tok_req.data_ptr<int>(); p.tok_len = tok_len.data_ptr<int>();
+  if (opt_ptr(head_bias) != nullptr) {
+    check_f32(*head_bias, "head_bias");
+    TORCH_CHECK(head_bias->numel() == p.H, "head_bias must be [H]");
+    p.slopes = head_bias->data_ptr<float>();
+  }
+  if (opt_ptr(turns_back) != nullptr) {
+    check_f32(*turns_back, "turns_back");
+    TORCH_CHECK(turns_back->dim() == 2 && turns_back->size(1) == 2 && 2 * turns_back->size(0) <= p.dv, "turns_back must be [n, 2], 2 n <= dv");
+    p.turns_back = turns_back->data_ptr<float>(); p.n_turn = static_cast<int>(turns_back->size(0)); p.interleaved = interleaved ? 1 : 0;
+  }
+  p.out = out.data_ptr();
+  p.block_size = static_cast<int>(block_size); p.max_blocks = static_cast<int>(block_table.size(1));
+  p.scale = static_cast<float>(scale); p.out_scale = 1.f; p.softcap = static_cast<float>(softcap);
+  c10::cuda::CUDAGuard g(q.device());
+  p.n_splits = 1;
+  Tensor ws;
+  if (block_table.size(0) == q.size(0) && q.size(0) > 0) {   // one token per sequence: a decoding batch
+    p.decode = 1;
+    const int64_t longest = max_len > 0 ? max_len : block_table.size(1) * block_size;      // unknown: what the tables can hold
+    p.n_splits = b200seq::window_attention_splits(p.H, p.G, p.n_tok, static_cast<int>(longest));
+    if (p.n_splits > 1) {
+      ws = torch::empty({q.size(0), p.H, p.n_splits, p.dv + 2}, q.options().dtype(at::kFloat));
+      p.ws = ws.data_ptr<float>();
+    }
+  }
+  TORCH_CHECK(b200seq::sigmoid_attention_paged(p, bf16, cur_stream()), "sigmoid_attention_paged: no kernel instance for heads ", p.H, " / ", p.G,
+              ", dims ", p.d, " / ", p.dv);
+  count(p.n_splits > 1 ? 2 : 1); check_last_error("sigmoid_attention_paged");
+}
+
+void gated_add_norm(Tensor x, c10::optional<Tensor> a, c10::optional<Tensor> ga, c10::optional<Tensor> bias_a, c10::optional<Tensor> b,
+                    c10::optional<Tensor> gb, c10::optional<Tensor> bias_b, const Tensor& w1, c10::optional<Tensor> w2, Tensor h1,
+                    c10::optional<Tensor> h2, double eps, bool center) {
+  check_f32(x, "x");
+  const bool bf16 = act_is_bf16(h1, "h1");
+  TORCH_CHECK(x.dim() == 2 && h1.is_contiguous() && h1.sizes() == x.sizes(), "x / h1 must be [rows, cols]");
+  b200seq::GatedNormArgs p{};
+  p.x = x.data_ptr<float>(); p.W = static_cast<int>(x.size(1)); p.center = center ? 1 : 0; p.eps = static_cast<float>(eps);
+  auto rows = [&](const c10::optional<Tensor>& t, const char* name, const void** ptr, int64_t* ld) {
+    if (opt_ptr(t) == nullptr) return;
+    check_act2(*t, h1, name);
+    TORCH_CHECK(t->sizes() == x.sizes(), name, " must be shaped like x");
+    *ptr = t->data_ptr(); *ld = t->stride(0);
+  };
+  auto vec = [&](const Tensor& t, const char* name) -> const void* {
+    TORCH_CHECK(t.is_cuda() && t.scalar_type() == h1.scalar_type() && t.is_contiguous() && t.numel() == x.size(1), name,
+                " must be a contiguous [cols] tensor in h1's dtype");
+    return t.data_ptr();
+  };
+  rows(a, "a", &p.a, &p.lda); rows(ga, "gate_a", &p.ga, &p.ldga); rows(b, "b", &p.b, &p.ldb); rows(gb, "gate_b", &p.gb, &p.ldgb);
+  TORCH_CHECK((p.ga == nullptr || p.a != nullptr) && (p.gb == nullptr || p.b != nullptr), "a gate without an addend");
+  if (opt_ptr(bias_a) != nullptr) p.bias_a = vec(*bias_a, "bias_a");
+  if (opt_ptr(bias_b) != nullptr) p.bias_b = vec(*bias_b, "bias_b");
+  p.w1 = vec(w1, "weight1"); p.h1 = h1.data_ptr();
+  if (opt_ptr(h2) != nullptr) {
+    TORCH_CHECK(opt_ptr(w2) != nullptr && h2->is_contiguous() && h2->sizes() == x.sizes() && h2->scalar_type() == h1.scalar_type(), "bad h2");
+    p.w2 = vec(*w2, "weight2"); p.h2 = h2->data_ptr();
+  }
+  c10::cuda::CUDAGuard g(x.device());
+  TORCH_CHECK(b200seq::gated_add_norm(p, static_cast<int>(x.size(0)), bf16, cur_stream()), "gated_add_norm: rows of ", p.W, " are too wide");
+  count(); check_last_error("gated_add_norm");
+}
+
+void head_rotary(const std::vector<Tensor>& x, const std::vector<c10::optional<Tensor>>& turns, const std::vector<c10::optional<Tensor>>& weight,
+                 const std::vector<c10::optional<Tensor>>& out, const std::vector<c10::optional<Tensor>>& pages,
+                 const std::vector<bool>& interleaved, const std::vector<double>& amplitude, const std::vector<bool>& back,
+                 const std::vector<bool>& rms, const std::vector<int64_t>& out_half, const std::vector<c10::optional<Tensor>>& table,
+                 const Tensor& positions, c10::optional<Tensor> slots, double eps) {
+  const size_t n = x.size();
+  TORCH_CHECK(n >= 1 && n <= 3 && turns.size() == n && weight.size() == n && out.size() == n && pages.size() == n && interleaved.size() == n &&
+              amplitude.size() == n && back.size() == n && rms.size() == n && out_half.size() == n && table.size() == n, "one to three parts");
+  const bool bf16 = act_is_bf16(x[0], "x");
+  const int64_t T = x[0].size(0);
+  TORCH_CHECK(positions.is_cuda() && positions.scalar_type() == at::kLong && positions.is_contiguous() && positions.numel() == T,
+              "positions must be int64 [T]");
+  b200seq::HeadRotaryArgs p{};
+  p.n_parts = static_cast<int>(n); p.eps = static_cast<float>(eps); p.positions = positions.data_ptr<int64_t>();
+  if (opt_ptr(slots) != nullptr) {
+    TORCH_CHECK(slots->is_cuda() && slots->scalar_type() == at::kLong && slots->is_contiguous() && slots->numel() == T, "slots must be int64 [T]");
+    p.slots = slots->data_ptr<int64_t>();
+  }
+  for (size_t k = 0; k < n; ++k) {
+    b200seq::RotPart& r = p.part[k];
+    TORCH_CHECK(x[k].is_cuda() && x[k].dim() == 3 && x[k].size(0) == T && x[k].stride(2) == 1 && x[k].scalar_type() == x[0].scalar_type(),
+                "x must be [T, heads, d] with unit inner stride, all of one dtype");
+    r.x = x[k].data_ptr(); r.ld_x = x[k].stride(0); r.hs_x = x[k].stride(1);
+    r.heads = static_cast<int>(x[k].size(1)); r.d = static_cast<int>(x[k].size(2));
+    r.interleaved = interleaved[k]; r.back = back[k]; r.rms = rms[k]; r.amplitude = static_cast<float>(amplitude[k]);
+    if (opt_ptr(turns[k]) != nullptr) {
+      check_f32(*turns[k], "turns");
+      TORCH_CHECK(turns[k]->dim() == 2 && turns[k]->size(1) == 2 && 2 * turns[k]->size(0) <= r.d, "turns must be [n, 2] with 2 n <= d");
+      r.turns = turns[k]->data_ptr<float>(); r.n_turn = static_cast<int>(turns[k]->size(0));
+    }
+    if (opt_ptr(table[k]) != nullptr) {
+      check_f32(*table[k], "table");
+      TORCH_CHECK(table[k]->numel() == T * r.n_turn * 2, "table must be [T, n, 2]");
+      r.table = table[k]->data_ptr<float>();
+    }
+    if (opt_ptr(weight[k]) != nullptr) {
+      TORCH_CHECK(weight[k]->scalar_type() == x[0].scalar_type() && weight[k]->is_contiguous() && weight[k]->numel() == r.d, "bad weight");
+      r.weight = weight[k]->data_ptr();
+    }
+    auto dst = [&](const Tensor& t, const char* name) {
+      TORCH_CHECK(t.is_cuda() && t.dim() == 3 && t.stride(2) == 1 && t.size(1) == r.heads && t.size(2) >= r.d && t.scalar_type() == x[0].scalar_type(),
+                  name, " must be [., heads, d] with unit inner stride in x's dtype");
+    };
+    if (opt_ptr(out[k]) != nullptr) {
+      dst(*out[k], "out");
+      TORCH_CHECK(out[k]->size(0) == T, "out must have one row per token");
+      r.out = out[k]->data_ptr(); r.ld_out = out[k]->stride(0); r.hs_out = out[k]->stride(1); r.d_out = static_cast<int>(out[k]->size(2));
+      r.out_half = static_cast<int>(out_half[k]);
+      TORCH_CHECK(r.out_half == 0 || (r.out_half >= r.d / 2 && r.out_half + r.d - r.d / 2 <= r.d_out), "bad out_half");
+    }
+    if (opt_ptr(pages[k]) != nullptr) {
+      dst(*pages[k], "pages");
+      TORCH_CHECK(p.slots != nullptr, "pages need slots");
+      r.pages = pages[k]->data_ptr(); r.ld_page = pages[k]->stride(0); r.hs_page = pages[k]->stride(1);
+    }
+  }
+  c10::cuda::CUDAGuard g(x[0].device());
+  TORCH_CHECK(b200seq::head_rotary(p, static_cast<int>(T), bf16, cur_stream()), "head_rotary: heads too wide");
+  count(); check_last_error("head_rotary");
+}
+
+void latent_head_assemble(const Tensor& q, const Tensor& k, const Tensor& k_rot, const Tensor& v, c10::optional<Tensor> turns, bool interleaved,
+                          double amplitude, const Tensor& positions, Tensor q_out, Tensor k_out, Tensor v_out) {
+  const bool bf16 = act_is_bf16(q, "q");
+  const auto dt = q.scalar_type();
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous() && k.scalar_type() == dt &&
+              v.scalar_type() == dt, "q / k / v must be contiguous [T, H, .] of one dtype");
+  check_act2(k_rot, q, "k_rot");
+  b200seq::LatentHeadArgs p{};
+  const int64_t T = q.size(0);
+  p.H = static_cast<int>(q.size(1)); p.d = static_cast<int>(k.size(2)); p.n = static_cast<int>(k_rot.size(1)); p.dv = static_cast<int>(v.size(2));
+  TORCH_CHECK(q.size(2) == p.d + p.n && k.size(0) == T && v.size(0) == T && k.size(1) == p.H && v.size(1) == p.H && k_rot.size(0) == T, "bad shapes");
+  TORCH_CHECK(positions.is_cuda() && positions.scalar_type() == at::kLong && positions.is_contiguous() && positions.numel() == T, "bad positions");
+  p.width = static_cast<int>(q_out.size(2));
+  for (const Tensor* o : {&q_out, &k_out, &v_out})
+    TORCH_CHECK(o->is_contiguous() && o->scalar_type() == dt && o->dim() == 3 && o->size(0) == T && o->size(1) == p.H && o->size(2) == p.width, "bad outputs");
+  TORCH_CHECK(p.width >= p.d + p.n && p.width >= p.dv, "outputs too narrow");
+  if (opt_ptr(turns) != nullptr) {
+    check_f32(*turns, "turns");
+    TORCH_CHECK(turns->dim() == 2 && turns->size(1) == 2 && 2 * turns->size(0) <= p.n, "turns must be [pairs, 2]");
+    p.turns = turns->data_ptr<float>(); p.n_turn = static_cast<int>(turns->size(0));
+  }
+  p.q = q.data_ptr(); p.k = k.data_ptr(); p.k_rot = k_rot.data_ptr(); p.ld_kr = k_rot.stride(0); p.v = v.data_ptr();
+  p.positions = positions.data_ptr<int64_t>(); p.q_out = q_out.data_ptr(); p.k_out = k_out.data_ptr(); p.v_out = v_out.data_ptr();
+  p.interleaved = interleaved ? 1 : 0; p.amplitude = static_cast<float>(amplitude);
+  c10::cuda::CUDAGuard g(q.device());
+  TORCH_CHECK(b200seq::latent_head_assemble(p, static_cast<int>(T), bf16, cur_stream()), "latent_head_assemble: too many pairs");
+  count(); check_last_error("latent_head_assemble");
+}
+
+void head_gate(const Tensor& o, const Tensor& gate, Tensor y) {
+  const bool bf16 = act_is_bf16(y, "y");
+  TORCH_CHECK(o.is_cuda() && o.dim() == 3 && o.stride(2) == 1 && y.is_contiguous() && y.sizes() == o.sizes() &&
+              (o.scalar_type() == y.scalar_type() || o.scalar_type() == at::kFloat), "o must be [T, H, dv], fp32 or in y's dtype");
+  check_act2(gate, y, "gate");
+  TORCH_CHECK(gate.size(0) == o.size(0) && gate.size(1) == o.size(1), "gate must be [T, H]");
+  c10::cuda::CUDAGuard g(o.device());
+  b200seq::head_gate(o.data_ptr(), o.scalar_type() == at::kFloat, o.stride(0), o.stride(1), gate.data_ptr(), gate.stride(0), y.data_ptr(),
+                     static_cast<int>(o.size(0)), static_cast<int>(o.size(1)), static_cast<int>(o.size(2)), bf16, cur_stream());
+  count(); check_last_error("head_gate");
+}
+
+void rglru_scan(const Tensor& u, const Tensor& w, const Tensor& bias, const Tensor& lam, c10::optional<Tensor> y_pre, const Tensor& cu,
+                const Tensor& rows, Tensor state, Tensor y, double decay_scale, int64_t max_len) {
+  const bool bf16 = act_is_bf16(u, "u");
+  check_act2(u, u, "u"); check_f32(state, "state"); check_i32(cu, "cu"); check_i32(rows, "rows");
+  b200seq::LruArgs p{};
+  p.n_tok = static_cast<int>(u.size(0)); p.C = static_cast<int>(u.size(1));
+  TORCH_CHECK(w.scalar_type() == u.scalar_type() && w.is_contiguous() && w.dim() == 4 && w.size(1) == 2 && w.size(2) == w.size(3) &&
+              w.size(0) * w.size(2) == p.C, "gate weights must be contiguous [B, 2, n, n] with B n channels");
+  p.n_blocks = static_cast<int>(w.size(0)); p.n = static_cast<int>(w.size(2));
+  TORCH_CHECK(bias.scalar_type() == u.scalar_type() && bias.is_contiguous() && bias.numel() == 2 * p.C && lam.scalar_type() == u.scalar_type() &&
+              lam.is_contiguous() && lam.numel() == p.C, "bad gate bias / lam");
+  TORCH_CHECK(state.dim() == 2 && state.size(1) == p.C && y.is_contiguous() && y.sizes() == u.sizes() && y.scalar_type() == u.scalar_type(), "bad state / y");
+  if (opt_ptr(y_pre) != nullptr) {
+    check_act2(*y_pre, u, "y_pre");
+    TORCH_CHECK(y_pre->sizes() == u.sizes(), "bad y_pre");
+    p.y_pre = y_pre->data_ptr(); p.ldy = y_pre->stride(0);
+  }
+  p.u = u.data_ptr(); p.ldu = u.stride(0); p.w = w.data_ptr(); p.bias = bias.data_ptr(); p.lam = lam.data_ptr();
+  p.cu = cu.data_ptr<int>(); p.rows = rows.data_ptr<int>(); p.state = state.data_ptr<float>(); p.y = y.data_ptr();
+  p.decay_scale = static_cast<float>(decay_scale);
+  const int R = static_cast<int>(rows.numel());
+  c10::cuda::CUDAGuard g(u.device());
+  p.max_runs = b200seq::lru_runs(static_cast<int>(max_len > 0 ? max_len : p.n_tok));
+  Tensor pre = torch::empty({u.size(0), 2, u.size(1)}, state.options()), ws;
+  p.pre = pre.data_ptr<float>();
+  if (p.max_runs > 1) {
+    ws = torch::empty({R, p.max_runs, u.size(1), 2}, state.options());
+    p.ws = ws.data_ptr<float>();
+  }
+  TORCH_CHECK(b200seq::rglru_scan(p, R, bf16, cur_stream()), "rglru_scan: too many gate blocks (", p.n_blocks, ")");
+  count(p.max_runs > 1 ? 4 : 2); check_last_error("rglru_scan");
+}
+
 void selective_scan(const Tensor& x, c10::optional<Tensor> z, const Tensor& B, const Tensor& Cm, const Tensor& dt_pre,
                     c10::optional<Tensor> dt_bias, const Tensor& A_log, const Tensor& D, const Tensor& cu, const Tensor& rows, Tensor state,
                     Tensor y, double out_scale) {
@@ -619,6 +852,12 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("head_rms_norm", &head_rms_norm);
   m.def("window_attention_paged", &window_attention_paged);
   m.def("selective_scan", &selective_scan);
+  m.def("sigmoid_attention_paged", &sigmoid_attention_paged);
+  m.def("gated_add_norm", &gated_add_norm);
+  m.def("head_rotary", &head_rotary);
+  m.def("latent_head_assemble", &latent_head_assemble);
+  m.def("head_gate", &head_gate);
+  m.def("rglru_scan", &rglru_scan);
   m.def("delta_rule_scan", &delta_rule_scan);
   m.def("mlstm_scan", &mlstm_scan);
   m.def("latent_attention_paged", &latent_attention_paged);

@@ -26,5 +26,14 @@ __device__ __forceinline__ float warp_max(float v) {
 }
 __device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + expf(-x)); }
 
+// Sine and cosine of pos * rate, the rate given in full turns as the sum of two floats: the product's rounding error is carried
+// along, so the fraction of a turn keeps fp32 accuracy for far positions.
+__device__ __forceinline__ void turn_angle(const float* rate, int pos, float* sn, float* cs) {
+  const float p = static_cast<float>(pos), hi = rate[0];
+  const float prod = __fmul_rn(p, hi), err = __fmaf_rn(p, hi, -prod);
+  const float frac = (prod - rintf(prod)) + __fmaf_rn(p, rate[1], err);
+  sincospif(2.f * frac, sn, cs);
+}
+
 }  // namespace dev
 }  // namespace b200seq

@@ -468,7 +468,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int h0 = (blockIdx.y * kAttnWarps + warp) * HGW;
   const int nh = max(0, min(HGW, p.H - h0));
-  const int r = p.r, len = p.tok_len[t];
+  const int r = p.r, rq = p.r + p.n_rot, len = p.tok_len[t];       // entries that are summed, entries that are scored
   const int per_split = (len + p.n_splits - 1) / p.n_splits;
   const int key_lo = blockIdx.z * per_split, key_hi = min(len, key_lo + per_split);
   const int* table = p.block_table + static_cast<int64_t>(p.tok_req[t]) * p.max_blocks;
@@ -480,7 +480,10 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
 #pragma unroll
     for (int e = 0; e < RPL; ++e) {
       const int i = lane + 32 * e;
-      qv[g][e] = (g < nh && i < r) ? ld(static_cast<const T*>(p.q) + (static_cast<int64_t>(t) * p.H + h0 + g) * r + i) * p.scale : 0.f;
+      qv[g][e] = 0.f;
+      if (g < nh && i < rq)
+        qv[g][e] = p.scale * (i < r ? ld(static_cast<const T*>(p.q) + (static_cast<int64_t>(t) * p.H + h0 + g) * r + i)
+                                    : ld(static_cast<const T*>(p.q_rot) + (static_cast<int64_t>(t) * p.H + h0 + g) * p.n_rot + i - r));
       acc[g][e] = 0.f;
     }
   }
@@ -490,12 +493,12 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
     __syncthreads();                                  // the previous tile has been consumed
     for (int j = warp; j < nk; j += kAttnWarps) {
       const int key = tile_lo + j;
-      const T* src = cache + (static_cast<int64_t>(table[key / p.block_size]) * p.block_size + key % p.block_size) * r;
+      const T* src = cache + (static_cast<int64_t>(table[key / p.block_size]) * p.block_size + key % p.block_size) * rq;
       if (p.vec_ok) {
-        for (int i = lane * VEC; i < r; i += 32 * VEC)
-          *reinterpret_cast<uint4*>(tile + j * r + i) = *reinterpret_cast<const uint4*>(src + i);
+        for (int i = lane * VEC; i < rq; i += 32 * VEC)
+          *reinterpret_cast<uint4*>(tile + j * rq + i) = *reinterpret_cast<const uint4*>(src + i);
       } else {
-        for (int i = lane; i < r; i += 32) tile[j * r + i] = src[i];
+        for (int i = lane; i < rq; i += 32) tile[j * rq + i] = src[i];
       }
     }
     __syncthreads();
@@ -512,7 +515,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
 #pragma unroll
           for (int e = 0; e < RPL; ++e) {
             const int i = lane + 32 * e;
-            const float c = i < r ? ld(tile + (j0 + kb) * r + i) : 0.f;
+            const float c = i < rq ? ld(tile + (j0 + kb) * rq + i) : 0.f;
 #pragma unroll
             for (int g = 0; g < HGW; ++g) sc[g][kb] = fmaf(qv[g][e], c, sc[g][kb]);
           }
@@ -540,7 +543,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
         const int i = lane + 32 * e;
         float c[kKeyBatch];
 #pragma unroll
-        for (int kb = 0; kb < kKeyBatch; ++kb) c[kb] = (i < r && j0 + kb < nk) ? ld(tile + (j0 + kb) * r + i) : 0.f;
+        for (int kb = 0; kb < kKeyBatch; ++kb) c[kb] = (i < r && j0 + kb < nk) ? ld(tile + (j0 + kb) * rq + i) : 0.f;
 #pragma unroll
         for (int g = 0; g < HGW; ++g) {
           float a = acc[g][e] * corr[g];
@@ -556,7 +559,8 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
     if (g >= nh) continue;
     const int64_t row = static_cast<int64_t>(t) * p.H + h0 + g;
     if (p.n_splits == 1) {
-      const float inv = 1.0f / l[g];
+      float inv = 1.0f / l[g];
+      if (p.gate != nullptr) inv *= sigmoidf_(ld(static_cast<const T*>(p.gate) + t * p.ldg + h0 + g));
 #pragma unroll
       for (int e = 0; e < RPL; ++e) {
         const int i = lane + 32 * e;
@@ -575,7 +579,9 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
 }
 
 // one warp per (token, head): merge the splits' (max, sum, weighted sum)
-__global__ void latent_attention_merge_kernel(const float* __restrict__ ws, float* __restrict__ out, int n_rows, int r, int n_splits) {
+template <typename T>
+__global__ void latent_attention_merge_kernel(const float* __restrict__ ws, float* __restrict__ out, int n_rows, int r, int n_splits,
+                                              const T* __restrict__ gate, int64_t ldg, int H) {
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (row >= n_rows) return;
   const int lane = threadIdx.x & 31;
@@ -587,84 +593,98 @@ __global__ void latent_attention_merge_kernel(const float* __restrict__ ws, floa
     const float mz = base[z * (r + 2)];
     den += (mz == -INFINITY ? 0.f : expf(mz - m_all)) * base[z * (r + 2) + 1];
   }
+  const float f = (gate != nullptr ? sigmoidf_(ld(gate + (row / H) * ldg + row % H)) : 1.f) / den;
   for (int i = lane; i < r; i += 32) {
     float num = 0.f;
     for (int z = 0; z < n_splits; ++z) {
       const float mz = base[z * (r + 2)];
       num += (mz == -INFINITY ? 0.f : expf(mz - m_all)) * base[z * (r + 2) + 2 + i];
     }
-    out[static_cast<int64_t>(row) * r + i] = num / den;
+    out[static_cast<int64_t>(row) * r + i] = num * f;
   }
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
 // router: one warp per token
 // ---------------------------------------------------------------------------------------------------------------------
-__global__ void group_limited_router_kernel(const float* __restrict__ logits, float* __restrict__ probs, bool* __restrict__ rmap,
-                                            int n_tok, int E, int topk, int G, int keep, int renorm) {
-  extern __shared__ float smem[];                   // per warp: scores [E], group best [G]
+__global__ void group_limited_router_kernel(const float* __restrict__ logits, const float* __restrict__ correction, float* __restrict__ probs,
+                                            bool* __restrict__ rmap, int n_tok, int E, int topk, int G, int keep, int renorm, int sigmoid,
+                                            int top2, float scale) {
+  extern __shared__ float smem[];                   // per warp: scores [E], choice scores [E], group marks [G], weights [E]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
   if (t >= n_tok) return;
-  float* s = smem + static_cast<int64_t>(warp) * (E + G);
-  float* gbest = s + E;
+  float* s = smem + static_cast<int64_t>(warp) * (3 * E + G);
+  float* choice = s + E;
+  float* w = choice + E;                            // weight of a chosen expert, -1 otherwise
+  float* mark = w + E;
   const float* z = logits + static_cast<int64_t>(t) * E;
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) { const float v = expf(z[e] - mx); s[e] = v; sum += v; }
-  sum = warp_sum(sum);
-  __syncwarp();
-  for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
+  if (sigmoid) {
+    for (int e = lane; e < E; e += 32) s[e] = sigmoidf_(z[e]);
+  } else {
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) { const float v = expf(z[e] - mx); s[e] = v; sum += v; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
+  }
+  for (int e = lane; e < E; e += 32) {
+    choice[e] = s[e] + (correction != nullptr ? correction[e] : 0.f);
+    w[e] = -1.f;
+  }
   __syncwarp();
   const int per = E / G;
   for (int g = lane; g < G; g += 32) {
-    float b = -1.f;
-    for (int e = g * per; e < (g + 1) * per; ++e) b = fmaxf(b, s[e]);
-    gbest[g] = b;
+    float b1 = -INFINITY, b2 = -INFINITY;           // the two best choice scores of the group
+    for (int e = g * per; e < (g + 1) * per; ++e) {
+      const float v = choice[e];
+      if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) { b2 = v; }
+    }
+    mark[g] = (top2 && per > 1) ? b1 + b2 : b1;
   }
   __syncwarp();
-  // drop all but the `keep` best groups: repeatedly take the best remaining group and mark it (score + 2 > 1)
-  for (int it = 0; it < keep; ++it) {
-    float bv = -1.f; int bi = 0x7fffffff;
-    for (int g = lane; g < G; g += 32) {
-      const float v = gbest[g];
-      if (v <= 1.5f && (v > bv || (v == bv && g < bi))) { bv = v; bi = g; }
+  // experts outside the `keep` best groups leave the choice: take the best remaining group again and again, then drop the rest
+  if (keep < G) {
+    uint32_t taken = 0;                             // bit j: group lane + 32 j of this lane is kept (G <= 1024)
+    for (int it = 0; it < keep; ++it) {
+      float bv = -INFINITY; int bi = 0x7fffffff;
+      for (int g = lane, j = 0; g < G; g += 32, ++j)
+        if (!(taken >> j & 1u) && (mark[g] > bv || (mark[g] == bv && g < bi))) { bv = mark[g]; bi = g; }
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, bv, o); const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+      }
+      if (bi < G && (bi & 31) == lane) taken |= 1u << (bi >> 5);
     }
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, bv, o); const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-    }
-    if (lane == 0 && bi < G) gbest[bi] += 2.f;
+    for (int g = lane, j = 0; g < G; g += 32, ++j)
+      if (!(taken >> j & 1u))
+        for (int e = g * per; e < (g + 1) * per; ++e) choice[e] = -INFINITY;
     __syncwarp();
   }
   float wsum = 0.f;
-  int chosen[32];                                   // topk <= 32 (checked on the host)
   for (int it = 0; it < topk; ++it) {
-    float bv = -1.f; int bi = 0x7fffffff;
+    float bv = -INFINITY; int bi = 0x7fffffff;
     for (int e = lane; e < E; e += 32) {
-      const float v = s[e];
-      if (v >= 0.f && gbest[e / per] > 1.5f && (v > bv || (v == bv && e < bi))) { bv = v; bi = e; }
+      const float v = choice[e];
+      if (v > bv || (v == bv && v != -INFINITY && e < bi)) { bv = v; bi = e; }
     }
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, bv, o); const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
     }
-    chosen[it] = bi;
     if (bi < E) {
-      wsum += bv;
-      if (lane == 0) { probs[static_cast<int64_t>(t) * E + bi] = bv; s[bi] = -1.f; }
+      wsum += s[bi];
+      __syncwarp();
+      if (lane == 0) { w[bi] = s[bi]; choice[bi] = -INFINITY; }
     }
     __syncwarp();
   }
-  if (lane == 0) {
-    const float inv = renorm ? 1.0f / (wsum + 1e-20f) : 1.0f;
-    for (int it = 0; it < topk; ++it)
-      if (chosen[it] < E) {
-        probs[static_cast<int64_t>(t) * E + chosen[it]] *= inv;
-        rmap[static_cast<int64_t>(t) * E + chosen[it]] = true;
-      }
+  const float f = (renorm ? 1.0f / (wsum + 1e-20f) : 1.0f) * scale;
+  for (int e = lane; e < E; e += 32) {
+    probs[static_cast<int64_t>(t) * E + e] = w[e] >= 0.f ? w[e] * f : 0.f;
+    rmap[static_cast<int64_t>(t) * E + e] = w[e] >= 0.f;
   }
 }
 
@@ -770,7 +790,7 @@ bool mlstm_scan(const MlstmArgs& p, int R, bool bf16, cudaStream_t s) {
 
 template <typename T, int RPL, int HGW>
 static bool launch_attn(const LatentAttnArgs& p, int n_tok, cudaStream_t s) {
-  const size_t smem = static_cast<size_t>(kKeyTile) * p.r * sizeof(T);
+  const size_t smem = static_cast<size_t>(kKeyTile) * (p.r + p.n_rot) * sizeof(T);
   auto kern = latent_attention_kernel<T, RPL, HGW>;
   if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
     return false;
@@ -778,7 +798,7 @@ static bool launch_attn(const LatentAttnArgs& p, int n_tok, cudaStream_t s) {
   kern<<<grid, kAttnWarps * 32, smem, s>>>(p);
   if (p.n_splits > 1) {
     const int rows = n_tok * p.H;
-    latent_attention_merge_kernel<<<(rows + 3) / 4, 128, 0, s>>>(p.ws, p.out, rows, p.r, p.n_splits);
+    latent_attention_merge_kernel<T><<<(rows + 3) / 4, 128, 0, s>>>(p.ws, p.out, rows, p.r, p.n_splits, static_cast<const T*>(p.gate), p.ldg, p.H);
   }
   return true;
 }
@@ -805,7 +825,7 @@ static bool dispatch_attn_hgw(const LatentAttnArgs& p, int hgw, int n_tok, cudaS
 template <typename T>
 static bool dispatch_attn(const LatentAttnArgs& p, int n_tok, cudaStream_t s) {
   int rpl, hgw;
-  attn_shape(p.H, p.r, &rpl, &hgw);
+  attn_shape(p.H, p.r + p.n_rot, &rpl, &hgw);
   switch (rpl) {
     case 2: return dispatch_attn_hgw<T, 2>(p, hgw, n_tok, s);
     case 4: return dispatch_attn_hgw<T, 4>(p, hgw, n_tok, s);
@@ -830,15 +850,15 @@ bool latent_attention_paged(const LatentAttnArgs& p, int n_tok, bool bf16, cudaS
   return bf16 ? dispatch_attn<__nv_bfloat16>(p, n_tok, s) : dispatch_attn<float>(p, n_tok, s);
 }
 
-bool group_limited_router(const float* logits, float* probs, bool* rmap, int n_tok, int E, int topk, int G, int keep, bool renorm,
-                          cudaStream_t s) {
+bool group_limited_router(const float* logits, const float* correction, float* probs, bool* rmap, int n_tok, int E, int topk, int G, int keep,
+                          bool renorm, bool sigmoid, bool top2, float scale, cudaStream_t s) {
   if (n_tok == 0) return true;
-  if (topk > 32 || G <= 0 || E % G != 0) return false;
+  if (topk > E || G <= 0 || E % G != 0 || keep < 1 || keep > G || G > 1024) return false;
   const int warps = 4;
-  const size_t smem = static_cast<size_t>(warps) * (E + G) * sizeof(float);
+  const size_t smem = static_cast<size_t>(warps) * (3 * E + G) * sizeof(float);
   if (smem > 48 * 1024) return false;
-  group_limited_router_kernel<<<(n_tok + warps - 1) / warps, warps * 32, smem, s>>>(logits, probs, rmap, n_tok, E, topk, G, keep,
-                                                                                   renorm ? 1 : 0);
+  group_limited_router_kernel<<<(n_tok + warps - 1) / warps, warps * 32, smem, s>>>(logits, correction, probs, rmap, n_tok, E, topk, G, keep, renorm,
+                                                                                    sigmoid, top2, scale);
   return true;
 }
 

@@ -36,8 +36,12 @@ struct LatentAttnArgs {
   const void* q;                  // [T, H, r]
   const void* cache;              // [slots, r]
   const int *block_table, *tok_req, *tok_len;
+  const void* q_rot;              // [T, H, n_rot] scored against columns r .. r + n_rot - 1 of the cache rows (nullptr: none)
+  const void* gate;               // [T, H] pre-activation of the per-head output gate, row stride ldg (nullptr: none)
+  int64_t ldg;
   float* out;                     // [T, H, r]
   float* ws;                      // [T, H, n_splits, r + 2] when n_splits > 1
+  int n_rot;                      // cache rows hold r + n_rot entries
   int H, r, block_size, max_blocks, n_splits;
   int vec_ok;                     // rows of the cache may be copied 16 bytes at a time
   float scale;
@@ -55,8 +59,9 @@ bool mlstm_scan(const MlstmArgs& p, int R, bool bf16, cudaStream_t s);
 bool latent_attention_paged(const LatentAttnArgs& p, int n_tok, bool bf16, cudaStream_t s);
 // key splits per query token for a batch of n_tok tokens whose longest context is max_len
 int latent_attention_splits(int H, int r, int n_tok, int max_len);
-bool group_limited_router(const float* logits, float* probs, bool* rmap, int n_tok, int E, int topk, int G, int keep, bool renorm,
-                          cudaStream_t s);
+// scores: softmax or (sigmoid) logistic; choice = score + correction (nullptr: none); groups rank by their best or (top2) two best
+bool group_limited_router(const float* logits, const float* correction, float* probs, bool* rmap, int n_tok, int E, int topk, int G, int keep,
+                          bool renorm, bool sigmoid, bool top2, float scale, cudaStream_t s);
 
 struct NormRopeArgs {
   const void *q, *k;              // [T, q_ch], [T, k_ch] with row strides ldq / ldk (elements)
@@ -157,6 +162,10 @@ struct WindowAttnArgs {
   float* ws;                      // [T, H, n_splits, dv + 2] when n_splits > 1
   int QB, HC;                     // filled by the launcher
   float scale, out_scale;
+  // logistic weights only (slopes then holds the bias per head)
+  float softcap;                  // 0: none
+  const float* turns_back;        // [n_turn, 2] turns per position (high, low part) of the result's pairs (nullptr: none)
+  int n_turn, interleaved;        // pairs (i, i + n_turn), or (2 i, 2 i + 1)
 };
 
 struct SelScanArgs {
@@ -176,6 +185,7 @@ void add_sinusoid(float* x, const int64_t* positions, const float* freq, int n_t
 void head_rms_norm(const void* x, int64_t ldx, const void* w, void* y, int n_tok, int heads, int d, float eps, bool bf16,
                    cudaStream_t s);
 bool window_attention_paged(const WindowAttnArgs& p, bool bf16, cudaStream_t s);
+bool sigmoid_attention_paged(const WindowAttnArgs& p, bool bf16, cudaStream_t s);
 // key splits for a batch of n_tok single-token sequences whose longest visible context is max_keys
 int window_attention_splits(int H, int G, int n_tok, int max_keys);
 bool selective_scan(const SelScanArgs& p, int R, bool bf16, cudaStream_t s);
@@ -201,5 +211,71 @@ void decay_gates(const void* a, int64_t lda, const void* b, int64_t ldb, const v
                  int64_t rows, int C, int H, bool bf16, cudaStream_t s);
 // y = gelu_tanh(g) * e
 void gelu_mul(const void* g, int64_t ldg, const void* e, int64_t lde, void* y, int64_t rows, int cols, bool bf16, cudaStream_t s);
+
+struct GatedNormArgs {
+  float* x;                       // [T, W] stream, updated in place
+  const void *a, *ga, *bias_a;    // addend [T, W], pre-activation of its gate [T, W] (nullptr: one), the gate's bias [W] (nullptr: none)
+  const void *b, *gb, *bias_b;
+  int64_t lda, ldga, ldb, ldgb;
+  const void *w1, *w2;            // [W] norm weights of the two readers
+  void *h1, *h2;                  // [T, W]; h2 nullptr: one reader
+  int W, center;                  // center 0: RMS norm
+  float eps;
+};
+bool gated_add_norm(const GatedNormArgs& p, int n_tok, bool bf16, cudaStream_t s);
+
+struct RotPart {
+  const void* x;                  // [T, heads, d] with row stride ld_x and head stride hs_x
+  int64_t ld_x, hs_x;
+  const float* turns;             // [n_turn, 2] turns per position (high, low part)
+  int n_turn, interleaved, back, rms;
+  float amplitude;
+  const void* weight;             // [d] (nullptr: none)
+  int heads, d, d_out;
+  int out_half;                   // > 0: the second half of a head starts at this column of the dense result
+  float* table;                   // [T, n_turn, 2]: receives cosine and sine of the turns (nullptr: none)
+  void* out;                      // dense result, columns without a value are zeroed (nullptr: none)
+  int64_t ld_out, hs_out;
+  void* pages;                    // cache, row slots[t] (nullptr: none)
+  int64_t ld_page, hs_page;
+  int shares_table;               // filled by the launcher
+};
+struct HeadRotaryArgs {
+  RotPart part[3];
+  const int64_t *positions, *slots;
+  int n_parts;
+  int max_d;                      // filled by the launcher
+  float eps;
+};
+bool head_rotary(HeadRotaryArgs p, int n_tok, bool bf16, cudaStream_t s);
+
+struct LatentHeadArgs {
+  const void *q, *k, *k_rot, *v;  // [T, H, d + n], [T, H, d], [T, n] with row stride ld_kr, [T, H, dv]
+  int64_t ld_kr;
+  const float* turns;             // [n_turn, 2]
+  const int64_t* positions;
+  void *q_out, *k_out, *v_out;    // [T, H, width]
+  int H, d, n, dv, width, n_turn, interleaved;
+  float amplitude;
+};
+bool latent_head_assemble(const LatentHeadArgs& p, int n_tok, bool bf16, cudaStream_t s);
+// y [T, H, dv] = o * sigmoid(gate[t, h]); o fp32 or in y's type with row stride ldo and head stride hso
+void head_gate(const void* o, bool o_f32, int64_t ldo, int64_t hso, const void* gate, int64_t ldg, void* y, int n_tok, int H, int dv, bool bf16,
+               cudaStream_t s);
+
+struct LruArgs {
+  const void *u, *y_pre;          // [T, C] with row strides (y_pre nullptr: the state itself is the result)
+  int64_t ldu, ldy;
+  const void *w, *bias, *lam;     // [B, 2, n, n] gate matrices [out, in], [B, 2, n], [C]
+  const int *cu, *rows;
+  float* state;                   // [rows, C]
+  void* y;                        // [T, C]
+  float* pre;                     // [T, 2, C] workspace of the gates' pre-activations
+  float* ws;                      // [R, max_runs, C, 2] when max_runs > 1
+  int n_tok, C, n_blocks, n, max_runs;
+  float decay_scale;
+};
+int lru_runs(int max_len);
+bool rglru_scan(const LruArgs& p, int R, bool bf16, cudaStream_t s);
 
 }  // namespace b200seq

@@ -563,6 +563,21 @@ def attention_varlen(q, k, v, cu_seqlens_q, cu_seqlens_kv=None, scale=None, caus
     return torch.cat(outs, dim=0)
 
 
+def sigmoid_attention(q, k, v, cu, max_len: int, scale: float, softcap: float = 0.0, head_bias=None, back_table=None,
+                      interleaved: bool = False, v_dim: Optional[int] = None):
+    """Causal attention with logistic weights over packed 16-bit prompts (csrc/sigmoid_attn_sm100.cu; CUDA only -- the paged form
+    ``ops.seqmix.sigmoid_attention_paged`` serves everything else).  ``q [T, H, D]``, ``k, v [T, G, D]`` with ``D`` 64 or 128, heads
+    padded with zeros; ``cu`` int32 ``[R + 1]`` on the device, ``max_len`` the longest sequence.  ``back_table [T, n, 2]``: cosine and
+    sine by which the pairs of a token's result are turned back, ``(2 i, 2 i + 1)`` when ``interleaved``, else ``(i, n + i)`` with
+    the second half of every value starting at column ``D / 2`` of ``v``.  Returns ``[T, H * v_dim]``."""
+    T, H, D = q.shape
+    dv = D if v_dim is None else v_dim
+    o = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
+    ext().sigmoid_attn_fwd(q, k, v, cu, None if head_bias is None else head_bias.float().contiguous(), back_table, o, float(scale),
+                           float(softcap), bool(interleaved), int(max_len))
+    return o.view(T, H * dv)
+
+
 # ---------------------------------------------------------------------------
 # (vocab-parallel) cross entropy on [rows, vocab_local] logits
 # ---------------------------------------------------------------------------

@@ -914,9 +914,13 @@ class HeadPart:
     ``turns [n, 2]`` (``rotary_turns``; ``None``: nothing turns), pairs ``(i, i + n)`` or ``interleaved`` ``(2 i, 2 i + 1)``,
     ``amplitude`` on cosine and sine, ``back`` for the negative angle; ``rms``: every head is divided by its root mean square
     after the rotation, times ``weight [d]`` if given.  ``out``: ``[T, H, d']`` with ``d' >= d`` (the columns from ``d`` on
-    become zero), row ``t`` at ``out[t]``; ``pages``: ``[slots, H, d]``, row ``t`` at ``pages[slots[t]]``; either may be absent."""
+    become zero; with ``out_half`` the second half of a head starts at that column instead, zeros between and behind), row ``t``
+    at ``out[t]``; ``pages``: ``[slots, H, d]``, row ``t`` at ``pages[slots[t]]``; either may be absent.  ``table [T, n, 2]`` (fp32,
+    optional) receives the cosines and sines."""
 
-    def __init__(self, x, turns=None, interleaved=False, amplitude=1.0, back=False, rms=False, weight=None, out=None, pages=None):
+    def __init__(self, x, turns=None, interleaved=False, amplitude=1.0, back=False, rms=False, weight=None, out=None, pages=None,
+                 out_half=0, table=None):
+        self.out_half, self.table = int(out_half), table
         self.x, self.turns, self.interleaved, self.amplitude, self.back = x, turns, bool(interleaved), float(amplitude), bool(back)
         self.rms, self.weight, self.out, self.pages = bool(rms), weight, out, pages
 
@@ -930,14 +934,18 @@ def head_rotary(parts: Sequence[HeadPart], positions: torch.Tensor, eps: float, 
         kernel_calls["head_rotary"] += 1
         ext().head_rotary([p.x for p in parts], [p.turns for p in parts], [p.weight for p in parts], [p.out for p in parts],
                           [p.pages for p in parts], [p.interleaved for p in parts], [p.amplitude for p in parts],
-                          [p.back for p in parts], [p.rms for p in parts], positions, slots, float(eps))
+                          [p.back for p in parts], [p.rms for p in parts], [p.out_half for p in parts], [p.table for p in parts],
+                          positions, slots, float(eps))
         return
     for p in parts:
         y = p.x.float().clone()
         if p.turns is not None:
             n = p.turns.shape[0]
             cs, sn = _turn_tables(p.turns, positions, p.amplitude)
-            cs, sn = cs.unsqueeze(1), (-sn if p.back else sn).unsqueeze(1)
+            sn = -sn if p.back else sn
+            if p.table is not None:
+                p.table.copy_(torch.stack([cs, sn], dim=-1))
+            cs, sn = cs.unsqueeze(1), sn.unsqueeze(1)
             a, b = (slice(0, 2 * n, 2), slice(1, 2 * n, 2)) if p.interleaved else (slice(0, n), slice(n, 2 * n))
             u, w = y[..., a].clone(), y[..., b].clone()
             y[..., a] = u * cs - w * sn
@@ -948,8 +956,12 @@ def head_rotary(parts: Sequence[HeadPart], positions: torch.Tensor, eps: float, 
                 y = y * p.weight.float()
         d = y.shape[-1]
         if p.out is not None:
-            p.out[..., :d] = y.to(p.out.dtype)
-            p.out[..., d:] = 0
+            half = d // 2 if p.out_half else d
+            if p.out.shape[-1] > d:
+                p.out.zero_()
+            p.out[..., :half] = y[..., :half].to(p.out.dtype)
+            if p.out_half:
+                p.out[..., p.out_half:p.out_half + d - half] = y[..., half:].to(p.out.dtype)
         if p.pages is not None:
             p.pages[slots] = y.to(p.pages.dtype)
 

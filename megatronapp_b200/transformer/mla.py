@@ -341,16 +341,17 @@ class RotaryLatentAttention(MegatronModule):
             pages, slots, positions = ctx.latent_pages(key, r + n, proj.dtype), ctx.write_slots, ctx.positions
         else:
             table, tok_req, tok_len = dense_pages(s, b, proj.device)
-            pages, slots, positions = proj.new_empty(T, r + n), torch.arange(T, device=proj.device), tok_len.long() - 1
+            pages, slots, positions = None, None, tok_len.long() - 1
         flash = ctx is not None and self._flash_prefill(proj, ctx)
         cq = proj.new_empty(T, 1, o0)
-        c_out = proj.new_empty(T, 1, r) if flash else None
-        kr_out = proj.new_empty(T, 1, n) if flash else None
+        dense = flash or ctx is None
+        c_out, kr_out = (proj.new_empty(T, 1, r), proj.new_empty(T, 1, n)) if dense else (None, None)
+        c_page, kr_page = (None, None) if pages is None else (pages[:, :r].unsqueeze(1), pages[:, r:].unsqueeze(1))
         rot = dict(turns=self.turns, interleaved=self.interleaved, amplitude=self.amplitude)
         seqmix.head_rotary([HeadPart(proj[:, :o0].unsqueeze(1), rms=True, weight=self.q_norm_weight, out=cq),
                             HeadPart(proj[:, o0:o0 + r].unsqueeze(1), rms=True, weight=self.kv_norm_weight, out=c_out,
-                                     pages=pages[:, :r].unsqueeze(1)),
-                            HeadPart(proj[:, o0 + r:o0 + r + n].unsqueeze(1), out=kr_out, pages=pages[:, r:].unsqueeze(1), **rot)],
+                                     pages=c_page),
+                            HeadPart(proj[:, o0 + r:o0 + r + n].unsqueeze(1), out=kr_out, pages=kr_page, **rot)],
                            positions, self.eps, slots)
         q, _ = self.linear_q_up_proj(cq[:, 0])
         q = q.view(T, nh, d + n)
@@ -370,6 +371,6 @@ class RotaryLatentAttention(MegatronModule):
             if ctx is not None:
                 o_lat = ctx.attend_latent(key, q_lat, None, self.softmax_scale, q_rot, gate)
             else:
-                o_lat = seqmix.latent_attention_paged(q_lat, pages, table, tok_req, tok_len, s, self.softmax_scale, 0, q_rot, gate)
+                o_lat = seqmix.latent_attention_paged(q_lat, torch.cat([c_out, kr_out], dim=-1)[:, 0], table, tok_req, tok_len, s, self.softmax_scale, 0, q_rot, gate)
             o = torch.einsum("thr,hvr->thv", o_lat.to(wv.dtype), wv)
         return self.linear_proj(unpacked_tokens(o.reshape(T, nh * dv), s, b))

@@ -90,21 +90,27 @@ class SigmoidAttention(MegatronModule):
             flash = self._flash_prefill(proj, ctx)
         else:
             table, tok_req, tok_len = dense_pages(s, b, proj.device)
-            kc, vc = proj.new_empty(T, self.nkv, self.d), proj.new_empty(T, self.nkv, self.dv)
-            slots = torch.arange(T, device=proj.device)
+            kc = vc = slots = None
             positions = tok_len.long() - 1
         width = (64 if max(self.d, self.dv) <= 64 else 128) if flash else self.d
         qr = proj.new_empty(T, self.nh, width)
-        kr, vr = (proj.new_empty(T, self.nkv, width), proj.new_empty(T, self.nkv, width)) if flash else (None, None)
+        kr = vr = None
+        if flash or ctx is None:
+            kr, vr = proj.new_empty(T, self.nkv, width), proj.new_empty(T, self.nkv, width if flash else self.dv)
+        half, back = 0, None
+        if flash and self.value_turns is not None:                      # what the tcgen05 kernel turns the result back by
+            half = 0 if self.interleaved else width // 2
+            back = torch.empty(T, self.value_turns.shape[0], 2, dtype=torch.float32, device=proj.device)
         kw = dict(turns=self.turns, interleaved=self.interleaved, amplitude=self.amplitude, rms=self.qk_norm)
         seqmix.head_rotary([HeadPart(q, out=qr, **kw), HeadPart(k, out=kr, pages=kc, **kw),
-                            HeadPart(v, self.value_turns, self.interleaved, out=vr, pages=vc)], positions, self.eps, slots)
+                            HeadPart(v, self.value_turns, self.interleaved, out=vr, pages=vc, out_half=half, table=back)],
+                           positions, self.eps, slots)
         if flash:
-            o = ops.sigmoid_attention(qr, kr, vr, ctx.packed.cu_host, self.scale, self.softcap, self.head_bias, self.value_turns,
+            o = ops.sigmoid_attention(qr, kr, vr, ctx.packed.cu, ctx.packed.max_len, self.scale, self.softcap, self.head_bias, back,
                                       self.interleaved, self.dv)
         elif ctx is not None:
             o = ctx.attend_sigmoid(key, qr, self.scale, self.softcap, self.head_bias, self.value_turns, self.interleaved)
         else:
-            o = seqmix.sigmoid_attention_paged(qr, kc, vc, table, tok_req, tok_len, s, self.scale, self.softcap, self.head_bias,
+            o = seqmix.sigmoid_attention_paged(qr, kr, vr, table, tok_req, tok_len, s, self.scale, self.softcap, self.head_bias,
                                                self.value_turns, self.interleaved)
         return self.out_proj(unpacked_tokens(o, s, b))
