@@ -4,7 +4,9 @@ with ``--serving-design lerorax`` the Lerorax design beside its closest existing
 head sizes, and the Lerorax kernels beside their like kernels; with ``--serving-design domasun`` the Domasun design beside its
 closest existing model, Lerorax (two mixers side by side on a paged attention and a recurrent memory), and its kernels
 beside their like kernels; with ``--serving-design nunosun`` the Nunosun design beside its closest existing model, Domasun
-(sliding-window attention beside a recurrent memory, mixtures of experts), and its kernels beside their like kernels.
+(sliding-window attention beside a recurrent memory, mixtures of experts), and its kernels beside their like kernels; with
+``--serving-design nasipel`` the Nasipel design beside its closest existing model, Zikunex (latent attention, recurrent mixers,
+group-limited mixtures of experts), and its kernels beside their like kernels.
 
 Two parts, random weights, bf16:
 
@@ -40,6 +42,14 @@ def _peaks():
             d = json.load(f)
         return float(d["hbm_gbs"]), "measured"
     return 6650.0, "fallback"
+
+
+def _tensor_peak():
+    p = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
+    if os.path.exists(p):
+        with open(p) as f:
+            return float(json.load(f)["bf16_tflops"])
+    return 1590.0
 
 
 def zikunex_config(s):
@@ -242,13 +252,15 @@ def serve_numbers(model, vocab, prompts, prompt_len, decoders, context, steps, w
 
 def _kernel_bench(device):
     """``(bench, out, roofline)``: ``bench(name, fn, bytes, flops, like)`` times ``fn`` alone (median of 5, an L2-sized buffer
-    rewritten before each) and records achieved rates and the fraction of the roofline in ``out``."""
+    rewritten before each) and records achieved rates and the fraction of the roofline in ``out``; ``tensor``: the flops run on
+    the tensor cores and are held against the measured cuBLAS bf16 rate."""
     hbm, how = _peaks()
+    mma_peak = _tensor_peak()
     fma_peak = 148 * 128 * 2 * 1.965e9 / 1e12        # fp32 TFLOP/s of the CUDA cores at the maximum clock
     flush = torch.empty(160 << 20, dtype=torch.uint8, device=device)
     out = {}
 
-    def bench(name, fn, nbytes, flops=0.0, like=None):
+    def bench(name, fn, nbytes, flops=0.0, like=None, tensor=False):
         for _ in range(3):
             fn()
         ts = []
@@ -263,11 +275,12 @@ def _kernel_bench(device):
         ms = sorted(ts)[len(ts) // 2]
         gbs = nbytes / ms / 1e6
         tfl = flops / ms / 1e9
-        frac = max(gbs / hbm, tfl / fma_peak if flops else 0.0)
+        peak = mma_peak if tensor else fma_peak
+        frac = max(gbs / hbm, tfl / peak if flops else 0.0)
         out[name] = {"ms": round(ms, 4), "GB/s": round(gbs, 1), "TFLOP/s": round(tfl, 2), "roofline_frac": round(frac, 3),
-                     "bound": "fma" if flops and tfl / fma_peak > gbs / hbm else "hbm", "like": like}
+                     "bound": ("tensor" if tensor else "fma") if flops and tfl / peak > gbs / hbm else "hbm", "like": like}
 
-    return bench, out, {"hbm_gbs": hbm, "fp32_fma_tflops": round(fma_peak, 1), "peaks": how}
+    return bench, out, {"hbm_gbs": hbm, "fp32_fma_tflops": round(fma_peak, 1), "bf16_tflops": mma_peak, "peaks": how}
 
 
 def kernel_numbers_lerorax(s, device):
@@ -540,6 +553,147 @@ def kernel_numbers_nunosun(s, device):
     return out, roof
 
 
+def nasipel_config(s):
+    """A Nasipel stack at the sizes of ``s``: logistic attention (a key / value head per four query heads), two recurrent blocks
+    as wide as the model with a gate block per head, latent attention whose heads are three quarters unrotated; every layer with
+    the mixture of experts of ``s``."""
+    H, d = s["heads"], s["dim"]
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    att = {"heads": H, "kv_heads": max(1, H // 4), "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 30.0, "rot": {"dims": d, "base": 10000.0}}
+    lru = {"width": s["width"], "blocks": H, "conv": 4}
+    rot = d // 4
+    lat = {"heads": H, "dim": d - rot, "rot_dim": rot, "vdim": d, "kv_rank": s["kv_rank"], "q_rank": s["q_rank"], "scale": d ** -0.5,
+           "rot": {"dims": rot, "base": 10000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    pattern = [("attention", att), ("rglru", lru), ("rglru", lru), ("latent_attention", lat)]
+    return {"architecture": "Nasipel", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5},
+            "layers": [{"type": pattern[i % 4][0], "mixer": dict(pattern[i % 4][1]), "mlp": moe} for i in range(s["layers"])]}
+
+
+def build_nasipel(s, device):
+    from .models.nasipel import NasipelConfig, NasipelModel
+    from .parallel import state as ps
+
+    if not ps.model_parallel_is_initialized():
+        ps.initialize_model_parallel(1, 1)
+    ncfg = NasipelConfig.from_dict(nasipel_config(s))
+    base = ncfg.base_transformer_config(torch.bfloat16, use_cpu_initialization=False)
+    return NasipelModel(ncfg, base).to(device).eval()
+
+
+def kernel_numbers_nasipel(s, device):
+    """The kernels of the Nasipel design and their like kernels: time, achieved bytes/s (or flop/s) and the fraction of the
+    roofline (measured copy bandwidth; for products on the tensor cores the measured cuBLAS rate, on the CUDA cores fp32 FMA)."""
+    from . import ops
+    from .ops import seqmix
+    from .ops.seqmix import HeadPart
+
+    bench, out, roof = _kernel_bench(device)
+    rn = lambda *sh, dtype=torch.float32: torch.randn(*sh, device=device, dtype=dtype)  # noqa: E731
+    H, d, W, r = s["heads"], s["dim"], s["width"], s["kv_rank"]
+    bf = torch.bfloat16
+    G, rot = max(1, H // 4), d // 4
+    # -- decode attention: 64 requests x 2048 cached tokens
+    R, L, bs = 64, 2048, 16
+    nblk = R * L // bs
+    table = torch.randperm(nblk, device=device).to(torch.int32).view(R, L // bs)
+    req = torch.arange(R, dtype=torch.int32, device=device)
+    lens = torch.full((R,), L, dtype=torch.int32, device=device)
+    kc, vc, q = rn(nblk * bs, G, d, dtype=bf), rn(nblk * bs, G, d, dtype=bf), rn(R, H, d, dtype=bf)
+    pb_ = torch.randn(H, device=device) - 4.0
+    turns = seqmix.rotary_turns(d, 10000.0, device=device)[0]
+    bench("sigmoid_attention_paged.decode", lambda: seqmix.sigmoid_attention_paged(q, kc, vc, table, req, lens, bs, d ** -0.5, 30.0, pb_, turns,
+                                                                                   False, L),
+          R * L * G * d * 4, flops=R * L * H * d * 4, like="paged_attention.decode")
+    if ops.ext().paged_attention_supported(d, H // G):
+        bench("paged_attention.decode", lambda: ops.ext().paged_attention(q, kc, vc, table, req, lens, bs, d ** -0.5, 1),
+              R * L * G * d * 4, flops=R * L * H * d * 4)
+    cache = rn(nblk * bs, r + rot, dtype=bf)
+    ql, qr, gate = rn(R, H, r, dtype=bf), rn(R, H, rot, dtype=bf), rn(R, H, dtype=bf)
+    bench("latent_attention_paged.decode (rotated part, gate)",
+          lambda: seqmix.latent_attention_paged(ql, cache, table, req, lens, bs, 0.05, L, qr, gate),
+          R * L * (r + rot) * 2, flops=R * L * H * (2 * r + rot) * 2, like="latent_attention_paged.decode")
+    cache0 = rn(nblk * bs, r, dtype=bf)
+    bench("latent_attention_paged.decode", lambda: seqmix.latent_attention_paged(ql, cache0, table, req, lens, bs, 0.05, L),
+          R * L * r * 2, flops=R * L * H * r * 4)
+    # -- prompts: 4 x 2048 tokens
+    n = 2048
+    T = 4 * n
+    cu = torch.tensor([0, n, 2 * n, 3 * n, T], dtype=torch.int32, device=device)
+    pos = torch.arange(n, device=device).repeat(4)
+    q4, k4, v4 = rn(T, H, d, dtype=bf), rn(T, G, d, dtype=bf), rn(T, G, d, dtype=bf)
+    tab = rn(T, d // 2, 2)
+    fl = 4 * n * (n + 1) / 2 * H * d * 4
+    bench("sigmoid_attention (tcgen05).prefill", lambda: ops.sigmoid_attention(q4, k4, v4, cu, n, d ** -0.5, 30.0, pb_, tab, False, d),
+          T * (H * 2 + G * 2) * d * 2, flops=fl, like="attn_fwd (tcgen05).prefill", tensor=True)
+    cuh = [0, n, 2 * n, 3 * n, T]
+    bench("attn_fwd (tcgen05).prefill", lambda: ops.attention_varlen(q4, k4, v4, (cuh, cuh), None, d ** -0.5, True, 0.0, False),
+          T * (H * 2 + G * 2) * d * 2, flops=fl, tensor=True)
+    table1 = torch.randperm(n // bs, device=device).to(torch.int32).view(1, -1)
+    req1 = torch.zeros(n, dtype=torch.int32, device=device)
+    len1 = torch.arange(1, n + 1, dtype=torch.int32, device=device)
+    bench("sigmoid_attention_paged.prefill (1 x 2048)",
+          lambda: seqmix.sigmoid_attention_paged(q4[:n], kc, vc, table1, req1, len1, bs, d ** -0.5, 30.0, pb_, turns),
+          n * (H * 2 + G * 2) * d * 2, flops=fl / 4, like="paged_attention.prefill (1 x 2048)")
+    if ops.ext().paged_attention_supported(d, H // G):
+        bench("paged_attention.prefill (1 x 2048)", lambda: ops.ext().paged_attention(q4[:n], kc, vc, table1, req1, len1, bs, d ** -0.5, 1),
+              n * (H * 2 + G * 2) * d * 2, flops=fl / 4)
+    q1, qr1 = rn(n, H, r, dtype=bf), rn(n, H, rot, dtype=bf)
+    g1 = rn(n, H, dtype=bf)
+    pairs = n * (n + 1) / 2
+    bench("latent_attention_paged.prefill (1 x 2048, rotated part, gate)",
+          lambda: seqmix.latent_attention_paged(q1, cache, table1, req1, len1, bs, 0.05, n, qr1, g1),
+          n * (r + rot) * 2 + n * H * r * 6, flops=pairs * H * (2 * r + rot) * 2, like="latent_attention_paged.prefill (1 x 2048)")
+    bench("latent_attention_paged.prefill (1 x 2048)", lambda: seqmix.latent_attention_paged(q1, cache0, table1, req1, len1, bs, 0.05, n),
+          n * r * 2 + n * H * r * 6, flops=pairs * H * r * 4)
+    # -- recurrent unit: decode (64 x 1) and prefill (4 x 2048), beside the minGRU scan over as many channels
+    C, B = W, H
+    nb = C // B
+    wg, bg, lam = rn(B, 2, nb, nb, dtype=bf) * nb ** -0.5, rn(B, 2, nb, dtype=bf), rn(C, dtype=bf) - 4.0
+    for tag, R_, m in (("decode", 64, 1), ("prefill", 4, 2048)):
+        T_ = R_ * m
+        pb = seqmix.PackedBatch([i * m for i in range(R_ + 1)], list(range(R_)), device)
+        u, pr = rn(T_, C, dtype=bf), rn(T_, 3 * C, dtype=bf)
+        S = torch.zeros(R_, C, device=device)
+        bench(f"rglru_scan.{tag}", lambda: seqmix.rglru_scan(u, wg, bg, lam, pr[:, :C], pb, S),
+              T_ * C * 6 + R_ * C * 8 + B * 2 * nb * nb * 2, flops=T_ * C * nb * 4, like=f"mingru_scan.{tag}", tensor=True)
+        bench(f"mingru_scan.{tag}", lambda: seqmix.mingru_scan(pr[:, :C], pr[:, C:2 * C], pr[:, 2 * C:], pb, S), T_ * C * 8 + R_ * C * 8)
+    # -- additions and norms, rotations, convolution, router over 8192 tokens
+    x = rn(T, W)
+    a, b, ga, gb = (rn(T, W, dtype=bf) for _ in range(4))
+    w = torch.ones(W, device=device, dtype=bf)
+    bench("gated_add_norm (two gated addends, two norms)", lambda: seqmix.gated_add_norm(x, a, ga, w, b, gb, w, w, w, 1e-5, bf),
+          T * W * (4 + 4 + 2 * 4 + 2 * 2), like="add_rms_norm")
+    bench("add_rms_norm", lambda: seqmix.add_rms_norm(x, a, w, 1e-5, bf), T * W * (4 + 4 + 2 + 2))
+    proj = rn(T, (H + 2 * G) * d, dtype=bf)
+    qo, ko, vo = rn(T, H, d, dtype=bf), rn(T, G, d, dtype=bf), rn(T, G, d, dtype=bf)
+    slots = torch.randperm(nblk * bs, device=device)[:T]
+    kw = dict(turns=turns, rms=True)
+    qv, kv_, vv = (proj[:, i0 * d:(i0 + h) * d].unflatten(1, (h, d)) for i0, h in ((0, H), (H, G), (H + G, G)))
+    bench("head_rotary (q, k, v; pages)", lambda: seqmix.head_rotary([HeadPart(qv, out=qo, **kw), HeadPart(kv_, out=ko, pages=kc, **kw),
+                                                                      HeadPart(vv, turns, out=vo, pages=vc)], pos, 1e-5, slots),
+          T * (H + 2 * G) * d * 4 + T * 2 * G * d * 2, like="gated_head_rms_norm")
+    o, gt, wn = rn(T, H, d), rn(T, H * d, dtype=bf), torch.ones(d, device=device, dtype=bf)
+    bench("gated_head_rms_norm", lambda: seqmix.gated_head_rms_norm(o, wn, gt, 1e-5, bf), T * H * d * (4 + 2 + 2))
+    ql4, kn4, vl4, kr4 = rn(T, H, d, dtype=bf), rn(T, H, d - rot, dtype=bf), rn(T, H, d, dtype=bf), rn(T, rot, dtype=bf)
+    tr = seqmix.rotary_turns(rot, 10000.0, device=device)[0]
+    oo = [rn(T, H, d, dtype=bf) for _ in range(3)]
+    bench("latent_head_assemble", lambda: seqmix.latent_head_assemble(ql4, kn4, kr4, vl4, tr, True, 1.0, pos, *oo), T * H * d * (2 * 6),
+          like="gated_head_rms_norm")
+    gh = rn(T, H, dtype=bf)
+    bench("head_gate", lambda: seqmix.head_gate(oo[0], gh, bf), T * H * d * 4, like="gated_head_rms_norm")
+    xc, wc, cb = rn(T, 2 * C, dtype=bf), rn(C, 4, dtype=bf), rn(C, dtype=bf)
+    pbc = seqmix.PackedBatch(cuh, [0, 1, 2, 3], device)
+    win = torch.zeros(4, 3, C, device=device, dtype=bf)
+    bench("causal_conv (bias)", lambda: seqmix.causal_conv(xc[:, C:], wc, pbc, win, bias=cb), T * C * 4, like="causal_conv_silu")
+    bench("causal_conv_silu", lambda: seqmix.causal_conv_silu(xc[:, C:], wc, pbc, win), T * C * 4)
+    lg, corr = rn(T, s["experts"]), rn(s["experts"])
+    bench("group_limited_router (logistic, correction, two best)",
+          lambda: seqmix.group_limited_router(lg, s["top"], 4, 2, True, "sigmoid", corr, "top2", 2.5), T * s["experts"] * 9, like="group_limited_router")
+    bench("group_limited_router", lambda: seqmix.group_limited_router(lg, s["top"], 4, 2), T * s["experts"] * 9)
+    return out, roof
+
+
 def kernel_numbers(s, device):
     """Every new kernel alone and its like kernel: time, achieved bytes/s (or flop/s) and the fraction of the roofline."""
     from . import ops
@@ -667,7 +821,8 @@ def run(args):
     pairs = {"zikunex": (("zikunex", build_zikunex), ("gpt_gqa_moe", build_gpt)),
              "lerorax": (("lerorax", build_lerorax), ("zikunex", build_zikunex)),
              "domasun": (("domasun", build_domasun), ("lerorax", build_lerorax)),
-             "nunosun": (("nunosun", build_nunosun), ("domasun", build_domasun))}[design]
+             "nunosun": (("nunosun", build_nunosun), ("domasun", build_domasun)),
+             "nasipel": (("nasipel", build_nasipel), ("zikunex", build_zikunex))}[design]
     with torch.no_grad():
         for name, build in pairs:
             t0 = time.time()
@@ -680,7 +835,7 @@ def run(args):
             torch.cuda.empty_cache()
         if not getattr(args, "serving_models_only", False):
             fn = {"zikunex": kernel_numbers, "lerorax": kernel_numbers_lerorax, "domasun": kernel_numbers_domasun,
-                  "nunosun": kernel_numbers_nunosun}[design]
+                  "nunosun": kernel_numbers_nunosun, "nasipel": kernel_numbers_nasipel}[design]
             res["kernels"], res["roofline"] = fn(s, dev)
     print(json.dumps(res), flush=True)
     return res
