@@ -71,7 +71,7 @@ def build_seq(verbose: bool = False, force: bool = False) -> Path:
     """``csrc/seqmix/*.cu`` + ``bindings_seq.cpp`` -> ``_C_seq.so`` (content-hashed like the main extension)."""
     BUILD.mkdir(exist_ok=True)
     src_dir = CSRC / "seqmix"
-    headers = sorted(src_dir.glob("*.h")) + sorted(src_dir.glob("*.cuh"))
+    headers = sorted(src_dir.glob("*.h")) + sorted(src_dir.glob("*.cuh")) + [CSRC / "common.cuh"]
     stamp_path = BUILD / "stamps_seq.json"
     stamps = json.loads(stamp_path.read_text()) if stamp_path.exists() else {}
     nvcc = _nvcc()

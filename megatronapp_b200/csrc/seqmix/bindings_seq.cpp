@@ -796,15 +796,29 @@ void rglru_scan(const Tensor& u, const Tensor& w, const Tensor& bias, const Tens
   p.decay_scale = static_cast<float>(decay_scale);
   const int R = static_cast<int>(rows.numel());
   c10::cuda::CUDAGuard g(u.device());
-  p.max_runs = b200seq::lru_runs(static_cast<int>(max_len > 0 ? max_len : p.n_tok));
-  Tensor pre = torch::empty({u.size(0), 2, u.size(1)}, state.options()), ws;
-  p.pre = pre.data_ptr<float>();
-  if (p.max_runs > 1) {
-    ws = torch::empty({R, p.max_runs, u.size(1), 2}, state.options());
+const int longest = static_cast<int>(max_len > 0 ? max_len : p.n_tok);
+  auto workspace = [&]() {
+    Tensor ws = torch::empty({R, p.max_runs, u.size(1), 2}, state.options());
     p.ws = ws.data_ptr<float>();
+    return ws;
+  };
+  if (longest == 1) {
+    TORCH_CHECK(b200seq::rglru_step(p, R, bf16, cur_stream()), "rglru_scan: unsupported sizes");
+    count();
+  } else if (bf16 && b200seq::rglru_chunked_supported(p, longest)) {
+    p.max_runs = b200seq::lru_chunks(longest);
+    Tensor ws = workspace();
+    TORCH_CHECK(b200seq::rglru_scan_chunked(p, R, cur_stream()), "rglru_scan: the chunked kernel could not be launched");
+    count(3);
+  } else {
+    p.max_runs = b200seq::lru_runs(longest);
+    Tensor pre = torch::empty({u.size(0), 2, u.size(1)}, state.options()), ws;
+    p.pre = pre.data_ptr<float>();
+    if (p.max_runs > 1) ws = workspace();
+    TORCH_CHECK(b200seq::rglru_scan(p, R, bf16, cur_stream()), "rglru_scan: too many gate blocks (", p.n_blocks, ")");
+    count(p.max_runs > 1 ? 4 : 2);
   }
-  TORCH_CHECK(b200seq::rglru_scan(p, R, bf16, cur_stream()), "rglru_scan: too many gate blocks (", p.n_blocks, ")");
-  count(p.max_runs > 1 ? 4 : 2); check_last_error("rglru_scan");
+  check_last_error("rglru_scan");
 }
 
 void selective_scan(const Tensor& x, c10::optional<Tensor> z, const Tensor& B, const Tensor& Cm, const Tensor& dt_pre,
@@ -858,6 +872,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("latent_head_assemble", &latent_head_assemble);
   m.def("head_gate", &head_gate);
   m.def("rglru_scan", &rglru_scan);
+  m.def("rglru_status", []() { return b200seq::rglru_chunked_status(); });
   m.def("delta_rule_scan", &delta_rule_scan);
   m.def("mlstm_scan", &mlstm_scan);
   m.def("latent_attention_paged", &latent_attention_paged);

@@ -803,20 +803,22 @@ static bool launch_attn(const LatentAttnArgs& p, int n_tok, cudaStream_t s) {
   return true;
 }
 
-// latent entries per lane (a power of two >= r / 32) and heads per warp: as many as fit 32 accumulators per lane, but no more
-// than it takes to spread the heads over the CTA's warps
+// latent entries per lane (the smallest instance >= r / 32: powers of two, and 10 and 18 for a power of two plus a rotated key part)
+// and heads per warp: as many as fit 36 accumulators per lane, but no more than it takes to spread the heads over the CTA's warps
 static void attn_shape(int H, int r, int* rpl, int* hgw) {
-  int e = 2;
-  while (e * 32 < r) e *= 2;
+  const int sizes[] = {2, 4, 8, 10, 16, 18, 32};
+  int e = 64;
+  for (int v : sizes)
+    if (v * 32 >= r) { e = v; break; }
   int g = 1;
-  while (g < 8 && g * 2 * e <= 32 && kAttnWarps * g < H) g *= 2;
+  while (g < 8 && g * 2 * e <= 36 && kAttnWarps * g < H) g *= 2;
   *rpl = e; *hgw = g;
 }
 
 template <typename T, int RPL>
 static bool dispatch_attn_hgw(const LatentAttnArgs& p, int hgw, int n_tok, cudaStream_t s) {
   if (hgw == 1) return launch_attn<T, RPL, 1>(p, n_tok, s);
-  if constexpr (RPL <= 16) { if (hgw == 2) return launch_attn<T, RPL, 2>(p, n_tok, s); }
+  if constexpr (RPL <= 18) { if (hgw == 2) return launch_attn<T, RPL, 2>(p, n_tok, s); }
   if constexpr (RPL <= 8) { if (hgw == 4) return launch_attn<T, RPL, 4>(p, n_tok, s); }
   if constexpr (RPL <= 4) { if (hgw == 8) return launch_attn<T, RPL, 8>(p, n_tok, s); }
   return false;
@@ -830,7 +832,9 @@ static bool dispatch_attn(const LatentAttnArgs& p, int n_tok, cudaStream_t s) {
     case 2: return dispatch_attn_hgw<T, 2>(p, hgw, n_tok, s);
     case 4: return dispatch_attn_hgw<T, 4>(p, hgw, n_tok, s);
     case 8: return dispatch_attn_hgw<T, 8>(p, hgw, n_tok, s);
+    case 10: return dispatch_attn_hgw<T, 10>(p, hgw, n_tok, s);
     case 16: return dispatch_attn_hgw<T, 16>(p, hgw, n_tok, s);
+    case 18: return dispatch_attn_hgw<T, 18>(p, hgw, n_tok, s);
     case 32: return dispatch_attn_hgw<T, 32>(p, hgw, n_tok, s);
     default: return false;
   }

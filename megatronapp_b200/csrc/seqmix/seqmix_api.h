@@ -277,5 +277,12 @@ struct LruArgs {
 };
 int lru_runs(int max_len);
 bool rglru_scan(const LruArgs& p, int R, bool bf16, cudaStream_t s);
+// one token per sequence: gates and recurrence in one kernel, no workspace
+bool rglru_step(const LruArgs& p, int R, bool bf16, cudaStream_t s);
+// 16-bit prompts through tcgen05; p.max_runs = lru_chunks(max_len), p.pre unused
+int lru_chunks(int max_len);
+bool rglru_chunked_supported(const LruArgs& p, int max_len);
+bool rglru_scan_chunked(const LruArgs& p, int R, cudaStream_t s);
+int rglru_chunked_status();       // 1: a kernel of this process gave up on a wait
 
 }  // namespace b200seq

@@ -288,6 +288,19 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const TI* __restrict__ o
   st(y + i, ld(o + t * ldo + h * hso + c) * sigmoidf_(ld(gate + t * ldg + h)));
 }
 
+// four columns per thread (dv a multiple of 4, aligned rows)
+template <typename TI, typename T>
+__global__ void __launch_bounds__(256) head_gate_vec_kernel(const TI* __restrict__ o, int64_t ldo, int64_t hso, const T* __restrict__ gate,
+                                                            int64_t ldg, T* __restrict__ y, int64_t total4, int H, int dv4) {
+  for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total4; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t th = i / dv4;
+    const int t = static_cast<int>(th / H), h = static_cast<int>(th - static_cast<int64_t>(t) * H), c = static_cast<int>(i - th * dv4) * 4;
+    const float g = sigmoidf_(ld(gate + t * ldg + h));
+    const float4 v = ld4(o + t * ldo + h * hso + c);
+    st4(y + i * 4, make_float4(v.x * g, v.y * g, v.z * g, v.w * g));
+  }
+}
+
 }  // namespace
 
 bool gated_add_norm(const GatedNormArgs& p, int n_tok, bool bf16, cudaStream_t s) {
@@ -345,6 +358,18 @@ void head_gate(const void* o, bool o_f32, int64_t ldo, int64_t hso, const void* 
   const int64_t total = static_cast<int64_t>(n_tok) * H * dv;
   if (total == 0) return;
   const unsigned blocks = static_cast<unsigned>((total + 255) / 256);
+  if (dv % 4 == 0 && ldo % 4 == 0 && hso % 4 == 0 && reinterpret_cast<uintptr_t>(o) % 16 == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0) {
+    const unsigned vb = static_cast<unsigned>(std::min<int64_t>((total / 4 + 255) / 256, 148 * 32));
+    SEQ_DISPATCH_T(bf16, {
+      if (o_f32)
+        head_gate_vec_kernel<float, T><<<vb, 256, 0, s>>>(static_cast<const float*>(o), ldo, hso, static_cast<const T*>(gate), ldg,
+                                                          static_cast<T*>(y), total / 4, H, dv / 4);
+      else
+        head_gate_vec_kernel<T, T><<<vb, 256, 0, s>>>(static_cast<const T*>(o), ldo, hso, static_cast<const T*>(gate), ldg, static_cast<T*>(y),
+                                                      total / 4, H, dv / 4);
+    });
+    return;
+  }
   SEQ_DISPATCH_T(bf16, {
     if (o_f32)
       head_gate_kernel<float, T><<<blocks, 256, 0, s>>>(static_cast<const float*>(o), ldo, hso, static_cast<const T*>(gate), ldg, static_cast<T*>(y),

@@ -157,7 +157,115 @@ __global__ void __launch_bounds__(kLruThreads) lru_apply_kernel(LruArgs p) {
   if (!CARRIED) *st_ = S;
 }
 
+// ---------------------------------------------------------------------------------------------------------------------
+// A decoding batch, one token per sequence: grid (blocks, 32-channel slices, groups of 16 sequences).  Lane = output channel, a warp
+// carries four sequences; both gates' rows of the slice and the sequences' inputs are staged 128 wide in shared memory, 16-byte loads where rows allow.
+// ---------------------------------------------------------------------------------------------------------------------
+constexpr int kStepSeq = 16, kStepK = 128, kStepWarps = 4, kStepPer = kStepSeq / kStepWarps;
+
+template <typename T>
+__global__ void __launch_bounds__(kStepWarps * 32) lru_step_kernel(LruArgs p, int R) {
+  __shared__ float2 sw[kStepK][33];                        // (recurrence, input) weight of [k][channel]
+  __shared__ __align__(16) float su[kStepSeq][kStepK];
+  __shared__ int tok[kStepSeq];                            // packed token of each sequence, -1: none
+  const int n = p.n, b = blockIdx.x, o0 = blockIdx.y * 32, r0 = blockIdx.z * kStepSeq;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* w = static_cast<const T*>(p.w) + static_cast<int64_t>(b) * 2 * n * n;
+  const T* u = static_cast<const T*>(p.u) + b * n;
+  if (threadIdx.x < kStepSeq) {
+    const int r = r0 + threadIdx.x;
+    tok[threadIdx.x] = (r < R && p.cu[r] < p.cu[r + 1]) ? p.cu[r] : -1;
+  }
+  float ar[kStepPer], ai[kStepPer];
+#pragma unroll
+  for (int j = 0; j < kStepPer; ++j) ar[j] = ai[j] = 0.f;
+  // what the epilogue needs is on its way while the gates are summed
+  __syncthreads();
+  const int o = o0 + lane, c = b * n + min(o, n - 1);
+  const bool live = o < n;
+  const T* bias = static_cast<const T*>(p.bias) + static_cast<int64_t>(b) * 2 * n + min(o, n - 1);
+  const float br = ld(bias), bi = ld(bias + n), rate = p.decay_scale * softplusf_(ld(static_cast<const T*>(p.lam) + c));
+  int t_[kStepPer];
+  float uv_[kStepPer], y_[kStepPer], s_[kStepPer];
+  float* st_[kStepPer];
+#pragma unroll
+  for (int j = 0; j < kStepPer; ++j) {
+    t_[j] = tok[warp * kStepPer + j];
+    uv_[j] = y_[j] = s_[j] = 0.f;
+    st_[j] = nullptr;
+    if (t_[j] >= 0) {
+      st_[j] = p.state + static_cast<int64_t>(p.rows[r0 + warp * kStepPer + j]) * p.C + c;
+      s_[j] = *st_[j];
+      uv_[j] = ld(static_cast<const T*>(p.u) + static_cast<int64_t>(t_[j]) * p.ldu + c);
+      if (p.y_pre != nullptr) y_[j] = ld(static_cast<const T*>(p.y_pre) + static_cast<int64_t>(t_[j]) * p.ldy + c);
+    }
+  }
+  for (int k0 = 0; k0 < n; k0 += kStepK) {
+    __syncthreads();
+    constexpr int V = 16 / sizeof(T);                      // lane = channel: the shared-memory stores of a step are conflict-free
+    if (n % V == 0 && reinterpret_cast<uintptr_t>(p.w) % 16 == 0) {
+#pragma unroll
+      for (int q = 0; q < kStepK / V / kStepWarps; ++q) {
+        const int k = (warp + q * kStepWarps) * V, o = o0 + lane;
+        union { uint4 raw; T v[V]; } wr, wi;
+        wr.raw = wi.raw = make_uint4(0u, 0u, 0u, 0u);
+        if (o < n && k0 + k < n) {
+          const T* src = w + static_cast<int64_t>(o) * n + k0 + k;
+          wr.raw = *reinterpret_cast<const uint4*>(src);
+          wi.raw = *reinterpret_cast<const uint4*>(src + static_cast<int64_t>(n) * n);
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) sw[k + e][lane] = make_float2(ld(&wr.v[e]), ld(&wi.v[e]));
+      }
+    } else {
+      for (int i = threadIdx.x; i < 32 * kStepK; i += kStepWarps * 32) {
+        const int o = i / kStepK, k = i % kStepK;
+        const bool in = o0 + o < n && k0 + k < n;
+        const int64_t at = static_cast<int64_t>(o0 + o) * n + k0 + k;
+        sw[k][o] = in ? make_float2(ld(w + at), ld(w + at + static_cast<int64_t>(n) * n)) : make_float2(0.f, 0.f);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < kStepSeq * kStepK / (kStepWarps * 32); ++q) {
+      const int i = threadIdx.x + q * kStepWarps * 32, r = i / kStepK, k = i % kStepK;
+      su[r][k] = (tok[r] >= 0 && k0 + k < n) ? ld(u + static_cast<int64_t>(tok[r]) * p.ldu + k0 + k) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 4
+    for (int k = 0; k < kStepK; k += 4) {
+      float2 wv[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) wv[e] = sw[k + e][lane];
+#pragma unroll
+      for (int j = 0; j < kStepPer; ++j) {
+        const float4 uv = *reinterpret_cast<const float4*>(&su[warp * kStepPer + j][k]);
+        ar[j] = fmaf(wv[0].x, uv.x, ar[j]); ai[j] = fmaf(wv[0].y, uv.x, ai[j]);
+        ar[j] = fmaf(wv[1].x, uv.y, ar[j]); ai[j] = fmaf(wv[1].y, uv.y, ai[j]);
+        ar[j] = fmaf(wv[2].x, uv.z, ar[j]); ai[j] = fmaf(wv[2].y, uv.z, ai[j]);
+        ar[j] = fmaf(wv[3].x, uv.w, ar[j]); ai[j] = fmaf(wv[3].y, uv.w, ai[j]);
+      }
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < kStepPer; ++j) {
+    if (!live || t_[j] < 0) continue;
+    float a, put;
+    lru_gates(ar[j] + br, ai[j] + bi, uv_[j], rate, &a, &put);
+    const float S = fmaf(a, s_[j], put);
+    *st_[j] = S;
+    st(static_cast<T*>(p.y) + static_cast<int64_t>(t_[j]) * p.C + c, p.y_pre != nullptr ? S * gelu_tanhf_(y_[j]) : S);
+  }
+}
+
 }  // namespace
+
+bool rglru_step(const LruArgs& p, int R, bool bf16, cudaStream_t s) {
+  if (R == 0 || p.n_tok == 0 || p.C == 0) return true;
+  const dim3 grid(p.n_blocks, (p.n + 31) / 32, (R + kStepSeq - 1) / kStepSeq);
+  if (grid.y > 65535 || grid.z > 65535) return false;
+  SEQ_DISPATCH_T(bf16, lru_step_kernel<T><<<grid, kStepWarps * 32, 0, s>>>(p, R));
+  return true;
+}
 
 int lru_runs(int max_len) { return max_len <= kLruRun ? 1 : (max_len + kLruRun - 1) / kLruRun; }
 

@@ -352,6 +352,7 @@ def test_recurrent_unit_over_runs_and_steps(C, B, dtype, device):
     got = seqmix.rglru_scan(pd[:, :C], D(w), D(bias), D(lam), pd[:, C + 8:], seqmix.PackedBatch(cu, [2, 0, 1], device), state)
     close(got.float(), torch.cat(wants), tol)
     assert float(state[3].abs().max()) == 0.0
+    assert device == "cpu" or seqmix.ext().rglru_status() == 0         # no bounded wait ran out
     whole = state[2].clone()
     state.zero_()
     outs, at = [], 0
