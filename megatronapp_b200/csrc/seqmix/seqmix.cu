@@ -578,29 +578,29 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
   }
 }
 
-// one warp per (token, head): merge the splits' (max, sum, weighted sum)
+// one CTA per (token, head): merge the splits' (max, sum, weighted sum); at most 64 splits
 template <typename T>
-__global__ void latent_attention_merge_kernel(const float* __restrict__ ws, float* __restrict__ out, int n_rows, int r, int n_splits,
-                                              const T* __restrict__ gate, int64_t ldg, int H) {
-  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (row >= n_rows) return;
-  const int lane = threadIdx.x & 31;
+__global__ void __launch_bounds__(128) latent_attention_merge_kernel(const float* __restrict__ ws, float* __restrict__ out, int r, int n_splits,
+                                                                     const T* __restrict__ gate, int64_t ldg, int H) {
+  __shared__ float share[64];                       // what a split's weighted sum counts for
+  const int row = blockIdx.x, lane = threadIdx.x & 31;
   const float* base = ws + static_cast<int64_t>(row) * n_splits * (r + 2);
-  float m_all = -INFINITY;
-  for (int z = 0; z < n_splits; ++z) m_all = fmaxf(m_all, base[z * (r + 2)]);
-  float den = 0.f;
-  for (int z = 0; z < n_splits; ++z) {
-    const float mz = base[z * (r + 2)];
-    den += (mz == -INFINITY ? 0.f : expf(mz - m_all)) * base[z * (r + 2) + 1];
+  if (threadIdx.x < 32) {
+    const bool has0 = lane < n_splits, has1 = lane + 32 < n_splits;
+    const float m0 = has0 ? base[lane * (r + 2)] : -INFINITY, m1 = has1 ? base[(lane + 32) * (r + 2)] : -INFINITY;
+    const float l0 = has0 ? base[lane * (r + 2) + 1] : 0.f, l1 = has1 ? base[(lane + 32) * (r + 2) + 1] : 0.f;
+    const float M = warp_max(fmaxf(m0, m1));
+    const float f0 = m0 == -INFINITY ? 0.f : expf(m0 - M), f1 = m1 == -INFINITY ? 0.f : expf(m1 - M);
+    const float f = (gate != nullptr ? sigmoidf_(ld(gate + (row / H) * ldg + row % H)) : 1.f) / warp_sum(l0 * f0 + l1 * f1);
+    share[lane] = f0 * f;
+    share[lane + 32] = f1 * f;
   }
-  const float f = (gate != nullptr ? sigmoidf_(ld(gate + (row / H) * ldg + row % H)) : 1.f) / den;
-  for (int i = lane; i < r; i += 32) {
+  __syncthreads();
+  for (int i = threadIdx.x; i < r; i += blockDim.x) {
     float num = 0.f;
-    for (int z = 0; z < n_splits; ++z) {
-      const float mz = base[z * (r + 2)];
-      num += (mz == -INFINITY ? 0.f : expf(mz - m_all)) * base[z * (r + 2) + 2 + i];
-    }
-    out[static_cast<int64_t>(row) * r + i] = num * f;
+#pragma unroll 4
+    for (int z = 0; z < n_splits; ++z) num = fmaf(share[z], base[z * (r + 2) + 2 + i], num);
+    out[static_cast<int64_t>(row) * r + i] = num;
   }
 }
 
@@ -798,7 +798,7 @@ static bool launch_attn(const LatentAttnArgs& p, int n_tok, cudaStream_t s) {
   kern<<<grid, kAttnWarps * 32, smem, s>>>(p);
   if (p.n_splits > 1) {
     const int rows = n_tok * p.H;
-    latent_attention_merge_kernel<T><<<(rows + 3) / 4, 128, 0, s>>>(p.ws, p.out, rows, p.r, p.n_splits, static_cast<const T*>(p.gate), p.ldg, p.H);
+    latent_attention_merge_kernel<T><<<rows, 128, 0, s>>>(p.ws, p.out, p.r, p.n_splits, static_cast<const T*>(p.gate), p.ldg, p.H);
   }
   return true;
 }

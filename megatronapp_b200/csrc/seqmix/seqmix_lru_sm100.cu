@@ -136,6 +136,12 @@ lru_chunk_kernel(const __grid_constant__ CUtensorMap map_u, const __grid_constan
     const int unit = (uc & 63) >> 3;
     const __nv_bfloat16* yp = static_cast<const __nv_bfloat16*>(p.y_pre) + (p.y_pre != nullptr ? static_cast<int64_t>(lo) * p.ldy + c : 0);
     __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.y) + static_cast<int64_t>(lo) * p.C + c;
+    __nv_bfloat16 ynext[16];                                       // one batch ahead of its use
+    auto fetch_y = [&](int t0) {
+#pragma unroll
+      for (int j = 0; j < 16; ++j) ynext[j] = yp[static_cast<int64_t>(min(t0 + j, n_tok - 1)) * p.ldy];
+    };
+    if (APPLY && p.y_pre != nullptr) fetch_y(0);
     for (int t0 = 0; t0 < n_tok; t0 += 16) {               // the same trip count for the whole CTA: TMEM loads are warp-wide
       uint32_t vr[16], vi[16];
       tmem_ld_32x16(row + t0, vr);
@@ -143,7 +149,8 @@ lru_chunk_kernel(const __grid_constant__ CUtensorMap map_u, const __grid_constan
       float yv[16];
       if (APPLY && p.y_pre != nullptr) {
 #pragma unroll
-        for (int j = 0; j < 16; ++j) yv[j] = __bfloat162float(yp[static_cast<int64_t>(min(t0 + j, n_tok - 1)) * p.ldy]);
+        for (int j = 0; j < 16; ++j) yv[j] = __bfloat162float(ynext[j]);
+        fetch_y(t0 + 16);
       }
       tmem_ld_wait();
       // the sixteen tokens' gates are independent of each other and of the state; tokens past the end keep the state as it is
