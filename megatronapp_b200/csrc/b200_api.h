@@ -237,6 +237,22 @@ int sigmoid_attn_fwd(const SigAttnArgs& a, cudaStream_t s);
 int sigmoid_attn_status();   // 1: a kernel of this process gave up on a wait
 const char* sigmoid_attn_last_error();
 
+struct WinAttnArgs {
+  const void *q, *k, *v;   // [T, H, d], [T, G, d], [T, G, d] contiguous, padded with zeros to d = 64 or 128
+  void* o;                 // [T, H, dv]
+  const int* cu;           // [n_seqs + 1]
+  const void* sink;        // [H] logit of a key without a value, in q's type (nullptr: none)
+  const void* gate;        // [T, H * dv] pre-activation of the output gate, in q's type, row stride ldg (nullptr: none)
+  int64_t ldg;
+  int n_tok, n_seqs, max_len, H, G, d, dv;
+  int window;              // a token sees itself and the window - 1 tokens before it (0: all)
+  float scale;
+  bool is_bf16;
+};
+int window_attn_fwd(const WinAttnArgs& a, cudaStream_t s);
+int window_attn_status();    // 1: a kernel of this process gave up on a wait
+const char* window_attn_last_error();
+
 // ---------------------------------------------------------------- comm
 void push_flags_barrier(uint32_t* const* peer_flags, int rank, int size, int slot, uint32_t epoch,
                         cudaStream_t s);

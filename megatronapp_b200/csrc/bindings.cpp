@@ -718,6 +718,35 @@ void sigmoid_attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const T
   TORCH_CHECK(rc == 0, "b200 sigmoid_attn_fwd failed: ", rc, " ", b200::sigmoid_attn_last_error());
   count();
 }
+// q [T, H, d], k / v [T, G, d] contiguous (d 64 or 128, zero-padded) -> o [T, H, dv]
+void window_attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& cu, const c10::optional<Tensor>& sink,
+                     const c10::optional<Tensor>& gate, Tensor o, double scale, int64_t window, int64_t max_len) {
+  c10::cuda::CUDAGuard guard(q.device());
+  for (const Tensor* t : {&q, &k, &v})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 3 && t->is_contiguous() && t->scalar_type() == q.scalar_type() && t->size(0) == q.size(0) &&
+                t->size(2) == q.size(2), "q / k / v must be contiguous [T, heads, d] of one dtype");
+  TORCH_CHECK(q.scalar_type() == at::kBFloat16 || q.scalar_type() == at::kHalf, "16-bit operands only");
+  TORCH_CHECK(k.size(1) == v.size(1), "k and v must have the same heads");
+  TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == at::kInt && cu.is_contiguous() && cu.numel() >= 1, "cu must be int32");
+  TORCH_CHECK(o.is_contiguous() && o.dim() == 3 && o.size(0) == q.size(0) && o.size(1) == q.size(1) && o.scalar_type() == q.scalar_type(), "bad o");
+  b200::WinAttnArgs a{};
+  a.q = q.data_ptr(); a.k = k.data_ptr(); a.v = v.data_ptr(); a.o = o.data_ptr(); a.cu = cu.data_ptr<int>();
+  a.n_tok = static_cast<int>(q.size(0)); a.n_seqs = static_cast<int>(cu.numel()) - 1; a.max_len = static_cast<int>(max_len);
+  a.H = static_cast<int>(q.size(1)); a.G = static_cast<int>(k.size(1)); a.d = static_cast<int>(q.size(2)); a.dv = static_cast<int>(o.size(2));
+  if (sink.has_value() && sink->defined()) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == q.scalar_type() && sink->is_contiguous() && sink->numel() == a.H, "sink must be [H] in q's dtype");
+    a.sink = sink->data_ptr();
+  }
+  if (gate.has_value() && gate->defined()) {
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == q.scalar_type() && gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == q.size(0) &&
+                gate->size(1) == a.H * a.dv, "gate must be [T, H * dv] in q's dtype");
+    a.gate = gate->data_ptr(); a.ldg = gate->stride(0);
+  }
+  a.scale = static_cast<float>(scale); a.window = static_cast<int>(window); a.is_bf16 = is_bf16(q);
+  int rc = b200::window_attn_fwd(a, cur_stream());
+  TORCH_CHECK(rc == 0, "b200 window_attn_fwd failed: ", rc, " ", b200::window_attn_last_error());
+  count();
+}
 std::vector<Tensor> attn_bwd(const Tensor& d_o, const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& o,
                              const Tensor& lse, double scale, bool causal, const c10::optional<Tensor>& dq_out,
                              const c10::optional<Tensor>& dk_out, const c10::optional<Tensor>& dv_out) {
@@ -1043,6 +1072,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("attn_fwd", &attn_fwd);
   m.def("sigmoid_attn_fwd", &sigmoid_attn_fwd);
   m.def("sigmoid_attn_status", []() { return b200::sigmoid_attn_status(); });
+  m.def("window_attn_fwd", &window_attn_fwd);
+  m.def("window_attn_status", []() { return b200::window_attn_status(); });
   m.def("attn_bwd", &attn_bwd);
   m.def("arena_alloc", &arena_alloc);
   m.def("arena_open", &arena_open);

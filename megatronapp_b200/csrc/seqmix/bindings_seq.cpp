@@ -164,7 +164,8 @@ void check_act2(const Tensor& t, const Tensor& like, const char* name) {   // [T
 }
 
 void latent_attention_paged(const Tensor& q, c10::optional<Tensor> q_rot, const Tensor& cache, const Tensor& block_table, const Tensor& tok_req,
-                            const Tensor& tok_len, c10::optional<Tensor> gate, Tensor out, int64_t block_size, double scale, int64_t max_len) {
+                            const Tensor& tok_len, c10::optional<Tensor> gate, Tensor out, int64_t block_size, double scale, int64_t max_len,
+                            int64_t window, c10::optional<Tensor> sink) {
   const bool bf16 = act_is_bf16(q, "q_lat");
   TORCH_CHECK(q.dim() == 3 && q.is_contiguous(), "q_lat must be contiguous [T, H, r]");
   b200seq::LatentAttnArgs p{};
@@ -183,6 +184,13 @@ void latent_attention_paged(const Tensor& q, c10::optional<Tensor> q_rot, const 
     TORCH_CHECK(gate->size(0) == q.size(0) && gate->size(1) == q.size(1), "gate must be [T, H]");
     p.gate = gate->data_ptr(); p.ldg = gate->stride(0);
   }
+  if (opt_ptr(sink) != nullptr) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == q.scalar_type() && sink->is_contiguous() && sink->numel() == q.size(1),
+                "sink must be [H] in q_lat's dtype");
+    p.sink = sink->data_ptr();
+  }
+  p.window = static_cast<int>(window);
+  if (window > 0) max_len = std::min(max_len, window);
   p.q = q.data_ptr(); p.cache = cache.data_ptr();
   p.block_table = block_table.data_ptr<int>(); p.tok_req = tok_req.data_ptr<int>(); p.tok_len = tok_len.data_ptr<int>();
   p.out = out.data_ptr<float>();
@@ -672,6 +680,35 @@ void gated_add_norm(Tensor x, c10::optional<Tensor> a, c10::optional<Tensor> ga,
   count(); check_last_error("gated_add_norm");
 }
 
+void squash_add(Tensor x, c10::optional<Tensor> a, c10::optional<Tensor> alpha_o, c10::optional<Tensor> wo, c10::optional<Tensor> bo,
+                c10::optional<Tensor> alpha_n, c10::optional<Tensor> wn, c10::optional<Tensor> bn, c10::optional<Tensor> h, double mult,
+                double x_scale) {
+  check_f32(x, "x");
+  TORCH_CHECK(x.dim() == 2, "x must be [rows, cols]");
+  b200seq::SquashArgs p{};
+  p.x = x.data_ptr<float>(); p.W = static_cast<int>(x.size(1)); p.mult = static_cast<float>(mult); p.x_scale = static_cast<float>(x_scale);
+  const Tensor* like = opt_ptr(h) != nullptr ? &*h : (opt_ptr(a) != nullptr ? &*a : nullptr);
+  const bool bf16 = like != nullptr && act_is_bf16(*like, "h");
+  auto vec = [&](const c10::optional<Tensor>& t, int64_t n, const char* name) -> const void* {
+    TORCH_CHECK(opt_ptr(t) != nullptr && t->is_cuda() && t->scalar_type() == like->scalar_type() && t->is_contiguous() && t->numel() == n, name,
+                " must be a contiguous tensor of ", n, " in the activations' dtype");
+    return t->data_ptr();
+  };
+  if (opt_ptr(a) != nullptr) {
+    check_act2(*a, *like, "a");
+    TORCH_CHECK(a->sizes() == x.sizes(), "a must be shaped like x");
+    p.a = a->data_ptr(); p.lda = a->stride(0);
+    if (opt_ptr(wo) != nullptr) { p.wo = vec(wo, p.W, "weight"); p.bo = vec(bo, p.W, "bias"); p.alpha_o = vec(alpha_o, 1, "alpha"); }
+  }
+  if (opt_ptr(h) != nullptr) {
+    TORCH_CHECK(h->is_contiguous() && h->sizes() == x.sizes(), "h must be contiguous and shaped like x");
+    p.h = h->data_ptr(); p.wn = vec(wn, p.W, "next weight"); p.bn = vec(bn, p.W, "next bias"); p.alpha_n = vec(alpha_n, 1, "next alpha");
+  }
+  c10::cuda::CUDAGuard g(x.device());
+  b200seq::squash_add(p, static_cast<int>(x.size(0)), bf16, cur_stream());
+  count(); check_last_error("squash_add");
+}
+
 void head_rotary(const std::vector<Tensor>& x, const std::vector<c10::optional<Tensor>>& turns, const std::vector<c10::optional<Tensor>>& weight,
                  const std::vector<c10::optional<Tensor>>& out, const std::vector<c10::optional<Tensor>>& pages,
                  const std::vector<bool>& interleaved, const std::vector<double>& amplitude, const std::vector<bool>& back,
@@ -737,8 +774,8 @@ void latent_head_assemble(const Tensor& q, const Tensor& k, const Tensor& k_rot,
                           double amplitude, const Tensor& positions, Tensor q_out, Tensor k_out, Tensor v_out) {
   const bool bf16 = act_is_bf16(q, "q");
   const auto dt = q.scalar_type();
-  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous() && k.scalar_type() == dt &&
-              v.scalar_type() == dt, "q / k / v must be contiguous [T, H, .] of one dtype");
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && k.is_contiguous() && v.is_contiguous() &&
+              k.scalar_type() == dt && v.scalar_type() == dt, "q / k / v must be [T, H, .] of one dtype, k and v contiguous, q with contiguous heads");
   check_act2(k_rot, q, "k_rot");
   b200seq::LatentHeadArgs p{};
   const int64_t T = q.size(0);
@@ -754,7 +791,7 @@ void latent_head_assemble(const Tensor& q, const Tensor& k, const Tensor& k_rot,
     TORCH_CHECK(turns->dim() == 2 && turns->size(1) == 2 && 2 * turns->size(0) <= p.n, "turns must be [pairs, 2]");
     p.turns = turns->data_ptr<float>(); p.n_turn = static_cast<int>(turns->size(0));
   }
-  p.q = q.data_ptr(); p.k = k.data_ptr(); p.k_rot = k_rot.data_ptr(); p.ld_kr = k_rot.stride(0); p.v = v.data_ptr();
+  p.q = q.data_ptr(); p.ld_q = q.stride(0); p.k = k.data_ptr(); p.k_rot = k_rot.data_ptr(); p.ld_kr = k_rot.stride(0); p.v = v.data_ptr();
   p.positions = positions.data_ptr<int64_t>(); p.q_out = q_out.data_ptr(); p.k_out = k_out.data_ptr(); p.v_out = v_out.data_ptr();
   p.interleaved = interleaved ? 1 : 0; p.amplitude = static_cast<float>(amplitude);
   c10::cuda::CUDAGuard g(q.device());
@@ -767,10 +804,11 @@ void head_gate(const Tensor& o, const Tensor& gate, Tensor y) {
   TORCH_CHECK(o.is_cuda() && o.dim() == 3 && o.stride(2) == 1 && y.is_contiguous() && y.sizes() == o.sizes() &&
               (o.scalar_type() == y.scalar_type() || o.scalar_type() == at::kFloat), "o must be [T, H, dv], fp32 or in y's dtype");
   check_act2(gate, y, "gate");
-  TORCH_CHECK(gate.size(0) == o.size(0) && gate.size(1) == o.size(1), "gate must be [T, H]");
+  const bool per_element = gate.size(1) == o.size(1) * o.size(2);
+  TORCH_CHECK(gate.size(0) == o.size(0) && (per_element || gate.size(1) == o.size(1)), "gate must be [T, H] or [T, H * dv]");
   c10::cuda::CUDAGuard g(o.device());
-  b200seq::head_gate(o.data_ptr(), o.scalar_type() == at::kFloat, o.stride(0), o.stride(1), gate.data_ptr(), gate.stride(0), y.data_ptr(),
-                     static_cast<int>(o.size(0)), static_cast<int>(o.size(1)), static_cast<int>(o.size(2)), bf16, cur_stream());
+  b200seq::head_gate(o.data_ptr(), o.scalar_type() == at::kFloat, o.stride(0), o.stride(1), gate.data_ptr(), gate.stride(0), per_element,
+                     y.data_ptr(), static_cast<int>(o.size(0)), static_cast<int>(o.size(1)), static_cast<int>(o.size(2)), bf16, cur_stream());
   count(); check_last_error("head_gate");
 }
 
@@ -869,6 +907,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("sigmoid_attention_paged", &sigmoid_attention_paged);
   m.def("gated_add_norm", &gated_add_norm);
   m.def("head_rotary", &head_rotary);
+  m.def("squash_add", &squash_add);
   m.def("latent_head_assemble", &latent_head_assemble);
   m.def("head_gate", &head_gate);
   m.def("rglru_scan", &rglru_scan);

@@ -469,14 +469,19 @@ __global__ void __launch_bounds__(kAttnWarps * 32) latent_attention_kernel(Laten
   const int h0 = (blockIdx.y * kAttnWarps + warp) * HGW;
   const int nh = max(0, min(HGW, p.H - h0));
   const int r = p.r, rq = p.r + p.n_rot, len = p.tok_len[t];       // entries that are summed, entries that are scored
-  const int per_split = (len + p.n_splits - 1) / p.n_splits;
-  const int key_lo = blockIdx.z * per_split, key_hi = min(len, key_lo + per_split);
+  const int first = p.window > 0 ? max(0, len - p.window) : 0;     // the first visible key
+  const int per_split = (len - first + p.n_splits - 1) / p.n_splits;
+  const int key_lo = first + blockIdx.z * per_split, key_hi = min(len, key_lo + per_split);
   const int* table = p.block_table + static_cast<int64_t>(p.tok_req[t]) * p.max_blocks;
   const T* cache = static_cast<const T*>(p.cache);
   float qv[HGW][RPL], acc[HGW][RPL], mx[HGW], l[HGW];
 #pragma unroll
   for (int g = 0; g < HGW; ++g) {
     mx[g] = -INFINITY; l[g] = 0.f;
+    if (p.sink != nullptr && blockIdx.z == 0 && g < nh) {  // one key of that score, without a value
+      mx[g] = ld(static_cast<const T*>(p.sink) + h0 + g);
+      l[g] = mx[g] > -INFINITY ? 1.f : 0.f;
+    }
 #pragma unroll
     for (int e = 0; e < RPL; ++e) {
       const int i = lane + 32 * e;

@@ -39,6 +39,8 @@ struct LatentAttnArgs {
   const void* q_rot;              // [T, H, n_rot] scored against columns r .. r + n_rot - 1 of the cache rows (nullptr: none)
   const void* gate;               // [T, H] pre-activation of the per-head output gate, row stride ldg (nullptr: none)
   int64_t ldg;
+  const void* sink;               // [H] logit of a key without a value in the softmax denominator, in q's type (nullptr: none)
+  int window;                     // > 0: only the last `window` cached tokens are visible; 0: all
   float* out;                     // [T, H, r]
   float* ws;                      // [T, H, n_splits, r + 2] when n_splits > 1
   int n_rot;                      // cache rows hold r + n_rot entries
@@ -57,7 +59,7 @@ void causal_conv_silu(const void* x, int64_t ldx, const void* w, const void* bia
 bool delta_rule_scan(const DeltaArgs& p, int R, bool bf16, cudaStream_t s);
 bool mlstm_scan(const MlstmArgs& p, int R, bool bf16, cudaStream_t s);
 bool latent_attention_paged(const LatentAttnArgs& p, int n_tok, bool bf16, cudaStream_t s);
-// key splits per query token for a batch of n_tok tokens whose longest context is max_len
+// key splits per query token for a batch of n_tok tokens with at most max_len visible keys
 int latent_attention_splits(int H, int r, int n_tok, int max_len);
 // scores: softmax or (sigmoid) logistic; choice = score + correction (nullptr: none); groups rank by their best or (top2) two best
 bool group_limited_router(const float* logits, const float* correction, float* probs, bool* rmap, int n_tok, int E, int topk, int G, int keep,
@@ -224,6 +226,18 @@ struct GatedNormArgs {
 };
 bool gated_add_norm(const GatedNormArgs& p, int n_tok, bool bf16, cudaStream_t s);
 
+struct SquashArgs {
+  float* x;                       // [T, W] stream: x <- x_scale * x + mult * N_o(a), N(z) = tanh(alpha z) * w + b
+  const void* a;                  // [T, W] addend with row stride lda (nullptr: none)
+  int64_t lda;
+  const void *wo, *bo, *alpha_o;  // N_o: [W], [W], scalar (wo nullptr: a enters as it is)
+  const void *wn, *bn, *alpha_n;  // N_n
+  void* h;                        // [T, W] N_n of the new x (nullptr: not wanted)
+  int W;
+  float x_scale, mult;
+};
+void squash_add(const SquashArgs& p, int n_tok, bool bf16, cudaStream_t s);
+
 struct RotPart {
   const void* x;                  // [T, heads, d] with row stride ld_x and head stride hs_x
   int64_t ld_x, hs_x;
@@ -250,8 +264,8 @@ struct HeadRotaryArgs {
 bool head_rotary(HeadRotaryArgs p, int n_tok, bool bf16, cudaStream_t s);
 
 struct LatentHeadArgs {
-  const void *q, *k, *k_rot, *v;  // [T, H, d + n], [T, H, d], [T, n] with row stride ld_kr, [T, H, dv]
-  int64_t ld_kr;
+  const void *q, *k, *k_rot, *v;  // [T, H, d + n] with row stride ld_q, [T, H, d], [T, n] with row stride ld_kr, [T, H, dv]
+  int64_t ld_q, ld_kr;
   const float* turns;             // [n_turn, 2]
   const int64_t* positions;
   void *q_out, *k_out, *v_out;    // [T, H, width]
@@ -259,9 +273,10 @@ struct LatentHeadArgs {
   float amplitude;
 };
 bool latent_head_assemble(const LatentHeadArgs& p, int n_tok, bool bf16, cudaStream_t s);
-// y [T, H, dv] = o * sigmoid(gate[t, h]); o fp32 or in y's type with row stride ldo and head stride hso
-void head_gate(const void* o, bool o_f32, int64_t ldo, int64_t hso, const void* gate, int64_t ldg, void* y, int n_tok, int H, int dv, bool bf16,
-               cudaStream_t s);
+// y [T, H, dv] = o * sigmoid(gate[t, h]) or, elementwise, o * sigmoid(gate[t, h * dv + c]); o fp32 or in y's type with row stride ldo and
+// head stride hso
+void head_gate(const void* o, bool o_f32, int64_t ldo, int64_t hso, const void* gate, int64_t ldg, bool elementwise, void* y, int n_tok, int H,
+               int dv, bool bf16, cudaStream_t s);
 
 struct LruArgs {
   const void *u, *y_pre;          // [T, C] with row strides (y_pre nullptr: the state itself is the result)

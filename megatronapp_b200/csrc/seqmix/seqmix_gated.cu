@@ -246,7 +246,7 @@ __global__ void __launch_bounds__(256) latent_head_assemble_kernel(LatentHeadArg
   }
   __syncthreads();
   const int d = p.d, n = p.n, W = p.width, np = p.n_turn;
-  const T* q = static_cast<const T*>(p.q) + t * p.H * (d + n);
+  const T* q = static_cast<const T*>(p.q) + t * p.ld_q;
   const T* k = static_cast<const T*>(p.k) + t * p.H * d;
   const T* v = static_cast<const T*>(p.v) + t * p.H * p.dv;
   const T* kr = static_cast<const T*>(p.k_rot) + t * p.ld_kr;
@@ -280,24 +280,31 @@ __global__ void __launch_bounds__(256) latent_head_assemble_kernel(LatentHeadArg
 
 template <typename TI, typename T>
 __global__ void __launch_bounds__(256) head_gate_kernel(const TI* __restrict__ o, int64_t ldo, int64_t hso, const T* __restrict__ gate,
-                                                        int64_t ldg, T* __restrict__ y, int64_t total, int H, int dv) {
+                                                        int64_t ldg, int elementwise, T* __restrict__ y, int64_t total, int H, int dv) {
   const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const int64_t th = i / dv, t = th / H;
   const int c = static_cast<int>(i - th * dv), h = static_cast<int>(th - t * H);
-  st(y + i, ld(o + t * ldo + h * hso + c) * sigmoidf_(ld(gate + t * ldg + h)));
+  st(y + i, ld(o + t * ldo + h * hso + c) * sigmoidf_(ld(gate + t * ldg + (elementwise ? h * dv + c : h))));
 }
 
 // four columns per thread (dv a multiple of 4, aligned rows)
 template <typename TI, typename T>
 __global__ void __launch_bounds__(256) head_gate_vec_kernel(const TI* __restrict__ o, int64_t ldo, int64_t hso, const T* __restrict__ gate,
-                                                            int64_t ldg, T* __restrict__ y, int64_t total4, int H, int dv4) {
+                                                            int64_t ldg, int elementwise, T* __restrict__ y, int64_t total4, int H, int dv4) {
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < total4; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t th = i / dv4;
     const int t = static_cast<int>(th / H), h = static_cast<int>(th - static_cast<int64_t>(t) * H), c = static_cast<int>(i - th * dv4) * 4;
-    const float g = sigmoidf_(ld(gate + t * ldg + h));
     const float4 v = ld4(o + t * ldo + h * hso + c);
-    st4(y + i * 4, make_float4(v.x * g, v.y * g, v.z * g, v.w * g));
+    float4 g;
+    if (elementwise) {
+      g = ld4(gate + t * ldg + h * dv4 * 4 + c);
+      g = make_float4(sigmoidf_(g.x), sigmoidf_(g.y), sigmoidf_(g.z), sigmoidf_(g.w));
+    } else {
+      const float f = sigmoidf_(ld(gate + t * ldg + h));
+      g = make_float4(f, f, f, f);
+    }
+    st4(y + i * 4, make_float4(v.x * g.x, v.y * g.y, v.z * g.z, v.w * g.w));
   }
 }
 
@@ -353,30 +360,28 @@ bool latent_head_assemble(const LatentHeadArgs& p, int n_tok, bool bf16, cudaStr
   return true;
 }
 
-void head_gate(const void* o, bool o_f32, int64_t ldo, int64_t hso, const void* gate, int64_t ldg, void* y, int n_tok, int H, int dv, bool bf16,
-               cudaStream_t s) {
+template <typename TI, typename T>
+static void launch_head_gate(const void* o, int64_t ldo, int64_t hso, const void* gate, int64_t ldg, bool elementwise, void* y, int64_t total, int H,
+                             int dv, cudaStream_t s) {
+  const TI* op = static_cast<const TI*>(o);
+  const T* gp = static_cast<const T*>(gate);
+  T* yp = static_cast<T*>(y);
+  const bool gate_ok = !elementwise || (ldg % 4 == 0 && reinterpret_cast<uintptr_t>(gate) % (4 * sizeof(T)) == 0);
+  if (dv % 4 == 0 && ldo % 4 == 0 && hso % 4 == 0 && reinterpret_cast<uintptr_t>(o) % 16 == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0 && gate_ok) {
+    const unsigned blocks = static_cast<unsigned>(std::min<int64_t>((total / 4 + 255) / 256, 148 * 32));
+    head_gate_vec_kernel<TI, T><<<blocks, 256, 0, s>>>(op, ldo, hso, gp, ldg, elementwise, yp, total / 4, H, dv / 4);
+  } else {
+    head_gate_kernel<TI, T><<<static_cast<unsigned>((total + 255) / 256), 256, 0, s>>>(op, ldo, hso, gp, ldg, elementwise, yp, total, H, dv);
+  }
+}
+
+void head_gate(const void* o, bool o_f32, int64_t ldo, int64_t hso, const void* gate, int64_t ldg, bool elementwise, void* y, int n_tok, int H,
+               int dv, bool bf16, cudaStream_t s) {
   const int64_t total = static_cast<int64_t>(n_tok) * H * dv;
   if (total == 0) return;
-  const unsigned blocks = static_cast<unsigned>((total + 255) / 256);
-  if (dv % 4 == 0 && ldo % 4 == 0 && hso % 4 == 0 && reinterpret_cast<uintptr_t>(o) % 16 == 0 && reinterpret_cast<uintptr_t>(y) % 16 == 0) {
-    const unsigned vb = static_cast<unsigned>(std::min<int64_t>((total / 4 + 255) / 256, 148 * 32));
-    SEQ_DISPATCH_T(bf16, {
-      if (o_f32)
-        head_gate_vec_kernel<float, T><<<vb, 256, 0, s>>>(static_cast<const float*>(o), ldo, hso, static_cast<const T*>(gate), ldg,
-                                                          static_cast<T*>(y), total / 4, H, dv / 4);
-      else
-        head_gate_vec_kernel<T, T><<<vb, 256, 0, s>>>(static_cast<const T*>(o), ldo, hso, static_cast<const T*>(gate), ldg, static_cast<T*>(y),
-                                                      total / 4, H, dv / 4);
-    });
-    return;
-  }
   SEQ_DISPATCH_T(bf16, {
-    if (o_f32)
-      head_gate_kernel<float, T><<<blocks, 256, 0, s>>>(static_cast<const float*>(o), ldo, hso, static_cast<const T*>(gate), ldg, static_cast<T*>(y),
-                                                        total, H, dv);
-    else
-      head_gate_kernel<T, T><<<blocks, 256, 0, s>>>(static_cast<const T*>(o), ldo, hso, static_cast<const T*>(gate), ldg, static_cast<T*>(y), total,
-                                                    H, dv);
+    if (o_f32) launch_head_gate<float, T>(o, ldo, hso, gate, ldg, elementwise, y, total, H, dv, s);
+    else launch_head_gate<T, T>(o, ldo, hso, gate, ldg, elementwise, y, total, H, dv, s);
   });
 }
 

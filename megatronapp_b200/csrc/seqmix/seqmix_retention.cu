@@ -235,6 +235,39 @@ __global__ void gelu_mul_kernel(const T* __restrict__ g, int64_t ldg, const T* _
   st(y + idx, act * ld(e + r * lde + c));
 }
 
+// four columns per thread, a row per blockIdx.y step (cols a multiple of 4, aligned rows)
+template <typename T> struct Quad;
+template <> struct Quad<float> {
+  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+};
+template <> struct Quad<__nv_bfloat16> {
+  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+  static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 r;
+    r.x = *reinterpret_cast<const uint32_t*>(&a); r.y = *reinterpret_cast<const uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = r;
+  }
+};
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+template <typename T>
+__global__ void __launch_bounds__(256) gelu_mul_vec_kernel(const T* __restrict__ g, int64_t ldg, const T* __restrict__ e, int64_t lde,
+                                                           T* __restrict__ y, int64_t rows, int cols) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (c >= cols) return;
+  for (int64_t r = blockIdx.y; r < rows; r += gridDim.y) {
+    const float4 z = Quad<T>::load(g + r * ldg + c), u = Quad<T>::load(e + r * lde + c);
+    Quad<T>::store(y + r * cols + c, make_float4(gelu_tanh(z.x) * u.x, gelu_tanh(z.y) * u.y, gelu_tanh(z.z) * u.z, gelu_tanh(z.w) * u.w));
+  }
+}
+
 // log_decay = -exp(A_log[head]) * softplus(a + dt_bias), beta = sigmoid(b): the gates of the delta rule from the projections'
 // pre-activations, fp32 out.  C decay channels per row, C / H per head.
 template <typename T>
@@ -307,6 +340,13 @@ void decay_gates(const void* a, int64_t lda, const void* b, int64_t ldb, const v
 void gelu_mul(const void* g, int64_t ldg, const void* e, int64_t lde, void* y, int64_t rows, int cols, bool bf16, cudaStream_t s) {
   const int64_t n = rows * cols;
   if (n == 0) return;
+  auto ok = [](const void* p, int64_t row) { return row % 4 == 0 && reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (ok(g, ldg) && ok(e, lde) && ok(y, cols)) {
+    const dim3 grid((cols / 4 + 255) / 256, static_cast<unsigned>(std::min<int64_t>(rows, 65535)));
+    SEQ_DISPATCH_T(bf16, gelu_mul_vec_kernel<T><<<grid, 256, 0, s>>>(static_cast<const T*>(g), ldg, static_cast<const T*>(e), lde,
+                                                                    static_cast<T*>(y), rows, cols));
+    return;
+  }
   SEQ_DISPATCH_T(bf16, gelu_mul_kernel<T><<<static_cast<unsigned>((n + 255) / 256), 256, 0, s>>>(
                            static_cast<const T*>(g), ldg, static_cast<const T*>(e), lde, static_cast<T*>(y), rows, cols));
 }

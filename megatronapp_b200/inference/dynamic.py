@@ -232,12 +232,14 @@ class DynamicInferenceContext:
         return self.latents[layer][self._write_slots]
 
     def attend_latent(self, layer: int, q_lat: torch.Tensor, c_new: Optional[torch.Tensor], scale: float,
-                      q_rot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                      q_rot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, window: int = 0,
+                      sink: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``q_lat [T, H, r]`` (queries carried into the latent space) against the latent pages of ``layer``.  ``c_new
         [T, r]`` are this step's latents, written into their pages first; a layer that shares another layer's latents
         passes ``None`` and names that layer (whose pages this step already holds), and so does a layer that has written
         ``latent_pages`` itself.  ``q_rot [T, H, n]`` scores against ``n`` further columns of the page rows, ``gate [T, H]``
-        (pre-activation) scales each head's result.  Returns the softmax-weighted sum of latents, fp32 ``[T, H, r]``."""
+        (pre-activation) scales each head's result; ``window`` limits the visible tokens to the last ones, ``sink [H]`` adds a key
+        without a value to each head's softmax.  Returns the softmax-weighted sum of latents, fp32 ``[T, H, r]``."""
         from ..ops import seqmix
 
         if c_new is not None:
@@ -246,7 +248,7 @@ class DynamicInferenceContext:
             raise RuntimeError(f"layer {layer} has written no latents for this step")
         self.kernel_calls += 1
         return seqmix.latent_attention_paged(q_lat, self.latents[layer], self._block_table, self._tok_req, self._tok_len,
-                                             self.block_size, scale, self._max_len, q_rot, gate)
+                                             self.block_size, scale, self._max_len, q_rot, gate, window, sink)
 
     def attend_mixed(self, layer: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float,
                      talk: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -266,22 +268,22 @@ class DynamicInferenceContext:
         return seqmix.mixed_attention_paged(q, kc, vc, self._block_table, self._tok_req, self._tok_len, self.block_size, scale,
                                             talk, gate, self._max_len)
 
-    def attend_window(self, layer: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, window: int = 0,
+    def attend_window(self, layer: int, q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], scale: float, window: int = 0,
                       slopes: Optional[torch.Tensor] = None, sink: bool = False, gate: Optional[torch.Tensor] = None,
                       out_scale: float = 1.0, dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Sliding-window grouped-query attention over the pages of cache ``layer``: ``q [T, H, d]``, new ``k [T, G, d]`` /
-        ``v [T, G, dv]`` (written into their pages first; ``v`` may be a strided view), a distance penalty per head
+        ``v [T, G, dv]`` (written into their pages first; ``v`` may be a strided view; both ``None`` for a layer that has filled its
+        ``kv_pages`` at ``write_slots`` itself), a distance penalty per head
         (``slopes [H]``) or an additive bias by distance (``dist_bias [L, H]``), an optional sink in the softmax denominator
         and a per-head output gate ``[T, H]`` (pre-activation) -> ``[T, H * dv]``.  A token sees the ``window`` last positions of its sequence (0: all).  fp32 and 16-bit caches."""
         from ..ops import seqmix
 
-        if layer not in self.kv:
-            n_slots = self.num_blocks * self.block_size
-            self.kv[layer] = (torch.zeros(n_slots, *k.shape[1:], dtype=k.dtype, device=k.device),
-                              torch.zeros(n_slots, *v.shape[1:], dtype=v.dtype, device=v.device))
-        kc, vc = self.kv[layer]
-        kc[self._write_slots] = k
-        vc[self._write_slots] = v
+        if k is None:
+            kc, vc = self.kv[layer]
+        else:
+            kc, vc = self.kv_pages(layer, k.shape[1:], v.shape[1:], k.dtype)
+            kc[self._write_slots] = k
+            vc[self._write_slots] = v
         self.kernel_calls += 1
         return seqmix.window_attention_paged(q, kc, vc, self._block_table, self._tok_req, self._tok_len, self.block_size, scale,
                                              window, slopes, sink, gate, out_scale, self._max_len, dist_bias)

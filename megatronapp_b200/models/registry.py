@@ -78,6 +78,13 @@ def _nasipel(path, params_dtype, device, **overrides):
     return load_model_dir(path, params_dtype, device, **overrides)
 
 
+@register_architecture("Dufitar")
+def _dufitar(path, params_dtype, device, **overrides):
+    from .dufitar.loader import load_model_dir
+
+    return load_model_dir(path, params_dtype, device, **overrides)
+
+
 @register_architecture("GPTModel")
 def _gpt(path, params_dtype, device, **overrides):
     """A GPT / Llama-style folder: ``config.json`` holds ``TransformerConfig`` fields under ``transformer`` plus

@@ -578,6 +578,20 @@ def sigmoid_attention(q, k, v, cu, max_len: int, scale: float, softcap: float = 
     return o.view(T, H * dv)
 
 
+def window_attention(q, k, v, cu, max_len: int, scale: float, window: int = 0, sink=None, gate=None, v_dim: Optional[int] = None):
+    """Causal sliding-window softmax attention over packed 16-bit prompts (csrc/window_attn_sm100.cu; CUDA only -- the paged forms in
+    ``ops.seqmix`` serve everything else).  ``q [T, H, D]``, ``k, v [T, G, D]`` with ``D`` 64 or 128, heads padded with zeros; ``cu``
+    int32 ``[R + 1]`` on the device, ``max_len`` the longest sequence.  A token sees itself and the ``window - 1`` tokens before it (0:
+    all).  ``sink [H]``: a key of that score without a value in every softmax of head ``h``; ``gate [T, H * v_dim]`` (pre-activation,
+    any row stride): the result is multiplied by its sigmoid.  Returns ``[T, H * v_dim]``."""
+    T, H, D = q.shape
+    dv = D if v_dim is None else v_dim
+    o = torch.empty(T, H, dv, dtype=q.dtype, device=q.device)
+    ext().window_attn_fwd(q, k, v, cu, sink, gate if (gate is None or gate.stride(1) == 1) else gate.contiguous(), o, float(scale), int(window),
+                          int(max_len))
+    return o.view(T, H * dv)
+
+
 # ---------------------------------------------------------------------------
 # (vocab-parallel) cross entropy on [rows, vocab_local] logits
 # ---------------------------------------------------------------------------

@@ -287,7 +287,8 @@ def mlstm_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_i: torch.T
 
 def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, tok_req: torch.Tensor,
                            tok_len: torch.Tensor, block_size: int, scale: float, max_len: int = 0,
-                           q_rot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                           q_rot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, window: int = 0,
+                           sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of every packed query token over the latents of its own sequence, in the latent space.
 
     ``q_lat [T, H, r]``: the query of head ``h`` already carried into the latent space (``W_uk,h^T q_h``), so that
@@ -299,7 +300,10 @@ def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table
 
     ``q_rot [T, H, n]``: a second query part against ``n`` further columns of the cache rows (``cache [num_slots, r + n]``, one
     key part shared by all heads): ``score = (q_lat . c + q_rot . k) * scale``; the weighted sum stays over the first ``r``
-    columns.  ``gate [T, H]`` (pre-activation) multiplies head ``h``'s result by its sigmoid."""
+    columns.  ``gate [T, H]`` (pre-activation) multiplies head ``h``'s result by its sigmoid.
+
+    ``window``: only the last ``window`` cached tokens (the query's own included) are visible, 0: all.  ``sink [H]`` (in ``q_lat``'s
+    dtype): head ``h``'s softmax denominator also contains ``exp(sink[h])``, a key without a value that ``scale`` does not touch."""
     T, H, r = q_lat.shape
     n_rot = 0 if q_rot is None else q_rot.shape[2]
     if cache.shape[1] != r + n_rot:
@@ -309,7 +313,7 @@ def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table
         o = torch.empty(T, H, r, dtype=torch.float32, device=q_lat.device)
         ext().latent_attention_paged(q_lat.contiguous(), None if q_rot is None else q_rot.contiguous(), cache, block_table, tok_req, tok_len,
                                      None if gate is None else (gate if gate.stride(1) == 1 else gate.contiguous()), o, int(block_size),
-                                     float(scale), int(max_len))
+                                     float(scale), int(max_len), int(window), None if sink is None else sink.contiguous())
         return o
     o = torch.empty(T, H, r, dtype=torch.float32)
     q = q_lat.float() if q_rot is None else torch.cat([q_lat.float(), q_rot.float()], dim=-1)
@@ -324,8 +328,14 @@ def latent_attention_paged(q_lat: torch.Tensor, cache: torch.Tensor, block_table
         slots = block_table[req[t]].long()[pos // block_size] * block_size + pos % block_size
         c = cache[slots].float()                                                        # [L, r + n]
         s = torch.einsum("thr,lr->thl", q[t:e + 1], c) * scale
-        vis = pos.view(1, 1, L) < torch.tensor(lens[t:e + 1]).view(-1, 1, 1)
-        o[t:e + 1] = torch.einsum("thl,lr->thr", torch.softmax(s.masked_fill(~vis, float("-inf")), -1), c[:, :r])
+        n_vis = torch.tensor(lens[t:e + 1]).view(-1, 1, 1)
+        vis = pos.view(1, 1, L) < n_vis
+        if window > 0:
+            vis = vis & (pos.view(1, 1, L) >= n_vis - window)
+        s = s.masked_fill(~vis, float("-inf"))
+        if sink is not None:                                                            # one more column, which has no value
+            s = torch.cat([s, sink.float().view(1, H, 1).expand(s.shape[0], H, 1)], dim=-1)
+        o[t:e + 1] = torch.einsum("thl,lr->thr", torch.softmax(s, -1)[..., :L], c[:, :r])
         t = e + 1
     if gate is not None:
         o = o * torch.sigmoid(gate.float()).unsqueeze(-1)
@@ -870,6 +880,30 @@ def gated_add_norm(x: torch.Tensor, a: Optional[torch.Tensor], gate_a: Optional[
 
 
 # ---------------------------------------------------------------------------
+# squashing norm without row statistics, fused with the residual addition around it
+# ---------------------------------------------------------------------------
+
+def squash_add(x: torch.Tensor, a: Optional[torch.Tensor], out_norm: Optional[Tuple], next_norm: Optional[Tuple], mult: float,
+               out_dtype: torch.dtype, x_scale: float = 1.0) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """``x`` fp32 ``[T, W]`` becomes ``x_scale * x + mult * N_o(a)`` in place; returned with ``N_n(x)`` in ``out_dtype`` (``next_norm =
+    None``: with ``None``).  A norm is a triple ``(alpha, weight [W], bias [W])`` with a scalar ``alpha``: ``N(z) = tanh(alpha z) *
+    weight + bias``, element by element (Zhu et al., "Transformers without Normalization").  ``a [T, W]`` may be absent;
+    ``out_norm = None`` adds it as it is.  All arithmetic is fp32."""
+    if x.is_cuda:
+        kernel_calls["squash_add"] += 1
+        h = torch.empty(x.shape, dtype=out_dtype, device=x.device) if next_norm is not None else None
+        no, nn_ = out_norm or (None, None, None), next_norm or (None, None, None)
+        ext().squash_add(x, a if (a is None or a.stride(1) == 1) else a.contiguous(), *no, *nn_, h, float(mult), float(x_scale))
+        return x, h
+    squash = lambda z, n: torch.tanh(n[0].float() * z) * n[1].float() + n[2].float()  # noqa: E731
+    if x_scale != 1.0:
+        x.mul_(x_scale)
+    if a is not None:
+        x.add_((a.float() if out_norm is None else squash(a.float(), out_norm)) * mult)
+    return x, None if next_norm is None else squash(x, next_norm).to(out_dtype)
+
+
+# ---------------------------------------------------------------------------
 # rotary positions of whole heads, with an optional norm, written where the consumer reads
 # ---------------------------------------------------------------------------
 
@@ -976,7 +1010,7 @@ def latent_head_assemble(q: torch.Tensor, k: torch.Tensor, k_rot: torch.Tensor, 
     n = k_rot.shape[1]
     if q.is_cuda:
         kernel_calls["latent_head_assemble"] += 1
-        ext().latent_head_assemble(q.contiguous(), k.contiguous(), k_rot if k_rot.stride(1) == 1 else k_rot.contiguous(), v.contiguous(), turns,
+        ext().latent_head_assemble(_rows3(q), k.contiguous(), k_rot if k_rot.stride(1) == 1 else k_rot.contiguous(), v.contiguous(), turns,
                                    bool(interleaved), float(amplitude), positions, q_out, k_out, v_out)
         return
     q_out.zero_(), k_out.zero_(), v_out.zero_()
@@ -986,8 +1020,8 @@ def latent_head_assemble(q: torch.Tensor, k: torch.Tensor, k_rot: torch.Tensor, 
 
 
 def head_gate(o: torch.Tensor, gate: Optional[torch.Tensor], out_dtype: torch.dtype) -> torch.Tensor:
-    """``o [T, H, dv]`` (unit inner stride): head ``h`` times ``sigmoid(gate[:, h])`` (``gate [T, H]`` pre-activation, any row
-    stride; ``None``: as it is) -> contiguous ``[T, H, dv]`` in ``out_dtype``."""
+    """``o [T, H, dv]`` (unit inner stride): head ``h`` times ``sigmoid(gate[:, h])`` (``gate [T, H]`` pre-activation) or, with ``gate
+    [T, H * dv]``, element by element (any row stride; ``None``: as it is) -> contiguous ``[T, H, dv]`` in ``out_dtype``."""
     if gate is None:
         return o.to(out_dtype).contiguous()
     if o.is_cuda:
@@ -995,7 +1029,9 @@ def head_gate(o: torch.Tensor, gate: Optional[torch.Tensor], out_dtype: torch.dt
         y = torch.empty(o.shape, dtype=out_dtype, device=o.device)
         ext().head_gate(o if o.stride(2) == 1 else o.contiguous(), gate if gate.stride(1) == 1 else gate.contiguous(), y)
         return y
-    return (o.float() * torch.sigmoid(gate.float()).unsqueeze(-1)).to(out_dtype).contiguous()
+    g = torch.sigmoid(gate.float())
+    g = g.unsqueeze(-1) if gate.shape[1] == o.shape[1] else g.unflatten(1, o.shape[1:])
+    return (o.float() * g).to(out_dtype).contiguous()
 
 
 # ---------------------------------------------------------------------------

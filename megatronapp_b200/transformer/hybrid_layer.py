@@ -1,8 +1,8 @@
 """Layers over an fp32 residual stream with an arbitrary sequence mixer, and the blocks that stack them: pre-norm
 (``ResidualF32Layer`` / ``ResidualF32Block``), norm on the sublayer's output (``OutputNormF32Layer`` /
 ``OutputNormF32Block``), several streams (``StreamLayer`` / ``StreamBlock``), one norm read by mixer and feed-forward side
-by side (``ParallelF32Layer`` / ``ParallelF32Block``), and side by side with a norm and a gate each (``DualNormF32Layer`` /
-``DualNormF32Block``), further down.
+by side (``ParallelF32Layer`` / ``ParallelF32Block``), side by side with a norm and a gate each (``DualNormF32Layer`` /
+``DualNormF32Block``), and a norm before and after each sublayer (``SandwichF32Layer`` / ``SandwichF32Block``), further down.
 
 ``x <- x + mixer(norm1(x));  x <- x + mlp(norm2(x))`` (the second half is absent for a layer without feed-forward).
 The stream ``x`` stays fp32 whatever the parameter dtype; every addition is fused into the norm that follows it
@@ -19,7 +19,7 @@ import torch.nn as nn
 
 from ..scan.tracer import scope as _scope
 from .module import MegatronModule
-from .norms import BranchPair, OutputRMSNormAdd, ResidualRMSNorm
+from .norms import BranchPair, OutputRMSNormAdd, ResidualRMSNorm, SquashNorm
 
 
 class ResidualF32Layer(MegatronModule):
@@ -441,3 +441,72 @@ class DualNormF32Block(MegatronModule):
                 break
             pending = layer(h1.view(shape), None if h2 is None else h2.view(shape), inference_context=inference_context, cache_index=k)
         return h1.view(shape) if self.final_norm_weight is not None else x2.view(shape)
+
+
+class SandwichF32Layer(MegatronModule):
+    """A norm before and after each sublayer, both additions scaled::
+
+        x <- x + m * norm1b(mixer(norm1(x)));   x <- x + m * norm2b(mlp(norm2(x)))
+
+    with ``SquashNorm`` norms and ``m = residual_mult``.  The stream ``x`` is fp32; an addition, the norm of its addend and the norm
+    that reads the new ``x`` are one kernel, so a layer receives ``(x, h)`` and returns ``(x, h_next)``.  ``cross_layer`` carries what
+    layers share within a step (latents, say) from one mixer to another."""
+
+    def __init__(self, config, layer_number: int, mixer: nn.Module, mlp: Optional[nn.Module] = None, residual_mult: float = 1.0):
+        super().__init__(config)
+        self.layer_number, self.residual_mult = layer_number, float(residual_mult)
+        W = config.hidden_size
+        self.mixer, self.mlp = mixer, mlp
+        self.input_norm, self.mixer_norm = SquashNorm(config, W), SquashNorm(config, W)
+        self.pre_mlp_norm = SquashNorm(config, W) if mlp is not None else None
+        self.mlp_norm = SquashNorm(config, W) if mlp is not None else None
+        if mlp is not None and hasattr(mlp, "set_layer_number"):
+            mlp.set_layer_number(layer_number)
+
+    def forward(self, x, h, inference_context=None, cross_layer=None, next_norm: Optional[SquashNorm] = None):
+        with _scope("transformer_layer", layer=self.layer_number):
+            out, bias = self.mixer(h, inference_context=inference_context, cross_layer=cross_layer)
+            if bias is not None:
+                out = out + bias
+            x, h = self.mixer_norm.add(x, out, self.residual_mult, next_norm if self.mlp is None else self.pre_mlp_norm)
+            if self.mlp is not None:
+                out, bias = self.mlp(h)
+                if bias is not None:
+                    out = out + bias
+                x, h = self.mlp_norm.add(x, out, self.residual_mult, next_norm)
+        return x, h
+
+
+class SandwichF32Block(MegatronModule):
+    """A stack of ``SandwichF32Layer`` followed by the final norm.  ``layer_builders[i](i)`` builds layer ``i``; ``input_scale``
+    multiplies the block's input (the embeddings) in the kernel of the first norm.  ``tap(layer, residual)`` receives the stream
+    after every layer."""
+
+    def __init__(self, config, layer_builders: List[Callable[[int], SandwichF32Layer]], post_process: bool = True, input_scale: float = 1.0):
+        super().__init__(config)
+        self.layers = nn.ModuleList([build(i) for i, build in enumerate(layer_builders)])
+        self.final_norm = SquashNorm(config, config.hidden_size) if post_process else None
+        self.input_scale = float(input_scale)
+        self.input_tensor = None
+        self.tap = None
+
+    def set_input_tensor(self, t):
+        self.input_tensor = t
+
+    def forward(self, hidden_states, inference_context=None):
+        first_stage = self.input_tensor is None
+        x = hidden_states if first_stage else self.input_tensor
+        if x.dtype != torch.float32:
+            x = x.float()
+        x = x.clone() if x.requires_grad else x.contiguous()           # the stream is updated in place
+        norms = [layer.input_norm for layer in self.layers] + [self.final_norm]
+        scale = self.input_scale if first_stage else 1.0
+        if norms[0] is None:                                            # an empty stage
+            return x * scale
+        x, h = norms[0](x, scale)
+        cross_layer = {}
+        for i, layer in enumerate(self.layers):
+            x, h = layer(x, h, inference_context=inference_context, cross_layer=cross_layer, next_norm=norms[i + 1])
+            if self.tap is not None:
+                self.tap(i, x)
+        return x if self.final_norm is None else h

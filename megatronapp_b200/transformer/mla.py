@@ -265,25 +265,30 @@ class LatentSelfAttention(MegatronModule):
 
 
 class RotaryLatentAttention(MegatronModule):
-    """Latent attention with a rotated key part shared by the heads, served from latent pages, with an optional output gate.
+    """Latent attention with a rotated key part shared by the heads, served from latent pages; optional: a low-rank query, a sliding
+    window, a sink in the softmax denominator, an output gate per head or per element, another layer's latents.
 
     Per token at position ``i`` (``R_i``: rotation by the position, optionally YaRN-scaled)::
 
-        q = W_uq norm(W_dq h), head by head [unrotated | rotated];   [c~ | k~] = W_dkv h;   c = norm(c~), k_r = R_i k~
-        score_h(j) = (q_n . W_uk,h c_j + (R_i q_r) . k_r,j) * scale;   o_h = sigmoid(W_g h)_h * sum_j softmax_j W_uv,h c_j
+        q = W_uq norm(W_dq h), or W_q h (``q_rank = None``), head by head [unrotated | rotated]
+        [c~ | k~] = W_dkv h;   c = norm(c~), k_r = R_i k~
+        score_h(j) = (q_n . W_uk,h c_j + (R_i q_r) . k_r,j) * scale,   0 <= i - j < window (0: all)
+        p_j = exp(score_h(j)) / (exp(sink_h) + sum_j exp(score_h(j)));   o_h = sigmoid(W_g h)_h * sum_j p_j W_uv,h c_j
 
-    Cached per token: one row ``[c | k_r]``.  Like ``LatentSelfAttention`` it never expands the cache: the unrotated query is
-    carried into the latent space (``W_uk,h^T q_n``) and one paged kernel scores it together with the rotated part against
-    the rows and sums the latents; ``W_uv,h`` follows.  Fresh 16-bit prompts with heads of at most 128 expand K and V from the
-    step's latents and run through the tcgen05 flash kernel, operands padded to its width.  The down projections and the gate are one fused input
-    projection ``[dq | dkv | g]``; the latent's norm, the two rotations and the page write are one kernel.  Angles, norm
-    statistics, scores and softmax are fp32."""
+    Cached per token: one row ``[c | k_r]``.  ``kv_source_layer`` names a layer whose rows (after norm and rotation) this layer reads
+    instead of a down projection of its own; it has its own queries, up projections, window, sink and gate.  Like
+    ``LatentSelfAttention`` it never expands the cache: the unrotated query is carried into the latent space (``W_uk,h^T q_n``) and
+    one paged kernel scores it together with the rotated part against the rows and sums the latents; ``W_uv,h`` follows.  Fresh
+    16-bit prompts with heads of at most 128 expand K and V from the step's latents and run through a tcgen05 kernel, operands padded
+    to its width.  The down projections and the gate are one fused input projection ``[dq | dkv | g]`` (``[q | dkv | g]``); the
+    latent's norm, the rotations and the page write are one kernel.  Angles, norm statistics, scores and softmax are fp32."""
 
     FLASH_PREFILL_MIN_TOKENS = 64
 
-    def __init__(self, config, layer_number: int, num_heads: int, qk_dim: int, rot_dim: int, v_dim: int, kv_rank: int, q_rank: int,
+    def __init__(self, config, layer_number: int, num_heads: int, qk_dim: int, rot_dim: int, v_dim: int, kv_rank: int, q_rank: Optional[int],
                  softmax_scale: float, rot_base: float = 10000.0, rot_scaling: Optional[dict] = None, rot_dims: Optional[int] = None,
-                 interleaved: bool = True, head_gate: bool = False, eps: Optional[float] = None):
+                 interleaved: bool = True, head_gate: bool = False, eps: Optional[float] = None, window: int = 0, sink: bool = False,
+                 element_gate: bool = False, kv_source_layer: Optional[int] = None):
         super().__init__(config)
         from ..ops import seqmix
         from ..parallel.tp_layers import ColumnParallelLinear, RowParallelLinear
@@ -292,85 +297,132 @@ class RotaryLatentAttention(MegatronModule):
         rot_dims = rot_dim if rot_dims is None else rot_dims
         if rot_dims % 2 or rot_dims > rot_dim:
             raise ValueError("latent attention: rot_dims must be even and at most rot_dim")
-        self.layer_number = layer_number
+        if head_gate and element_gate:
+            raise ValueError("latent attention: one output gate, per head or per element")
+        if kv_source_layer is not None and not 0 <= kv_source_layer < layer_number:
+            raise ValueError(f"layer {layer_number} cannot read the latents of layer {kv_source_layer}")
+        self.layer_number, self.kv_source_layer = layer_number, kv_source_layer
         self.nh, self.qk_dim, self.rot_dim, self.v_dim = num_heads, qk_dim, rot_dim, v_dim
         self.kv_rank, self.q_rank, self.interleaved = kv_rank, q_rank, bool(interleaved)
-        self.softmax_scale = float(softmax_scale)
+        self.softmax_scale, self.window = float(softmax_scale), int(window)
         self.eps = config.layernorm_epsilon if eps is None else eps
-        self.g_ch = num_heads if head_gate else 0
+        self.q_ch = num_heads * (qk_dim + rot_dim) if q_rank is None else q_rank
+        self.c_ch = kv_rank + rot_dim if kv_source_layer is None else 0
+        self.element_gate = bool(element_gate)
+        self.g_ch = num_heads if head_gate else num_heads * v_dim if element_gate else 0
         col = dict(config=config, init_method=config.init_method, bias=False, skip_bias_add=False, gather_output=False)
-        self.in_proj = ColumnParallelLinear(config.hidden_size, q_rank + kv_rank + rot_dim + self.g_ch, **col)
-        self.q_norm_weight = ResidualRMSNorm(config, q_rank, self.eps).weight
-        self.kv_norm_weight = ResidualRMSNorm(config, kv_rank, self.eps).weight
-        self.linear_q_up_proj = ColumnParallelLinear(q_rank, num_heads * (qk_dim + rot_dim), **col)
+        self.in_proj = ColumnParallelLinear(config.hidden_size, self.q_ch + self.c_ch + self.g_ch, **col)
+        if q_rank is not None:
+            self.q_norm_weight = ResidualRMSNorm(config, q_rank, self.eps).weight
+            self.linear_q_up_proj = ColumnParallelLinear(q_rank, num_heads * (qk_dim + rot_dim), **col)
+        if kv_source_layer is None:
+            self.kv_norm_weight = ResidualRMSNorm(config, kv_rank, self.eps).weight
         self.linear_k_up_proj = ColumnParallelLinear(kv_rank, num_heads * qk_dim, **col)
         self.linear_v_up_proj = ColumnParallelLinear(kv_rank, num_heads * v_dim, **col)
-        turns, self.amplitude = seqmix.rotary_turns(rot_dims, rot_base, rot_scaling, self.in_proj.weight.device)
+        dev = self.in_proj.weight.device
+        self.sink = torch.nn.Parameter(torch.zeros(num_heads, dtype=config.params_dtype, device=dev)) if sink else None
+        turns, self.amplitude = seqmix.rotary_turns(rot_dims, rot_base, rot_scaling, dev)
         self.register_buffer("turns", turns, persistent=False)
         self.linear_proj = RowParallelLinear(num_heads * v_dim, config.hidden_size, config=config, init_method=config.output_layer_init_method,
                                              bias=False, input_is_parallel=True, skip_bias_add=True)
 
     def segments(self):
-        """Row counts of the ``[dq | dkv | g]`` segments of ``in_proj`` (an absent gate is left out)."""
-        return [(n, c) for n, c in (("dq", self.q_rank), ("dkv", self.kv_rank + self.rot_dim), ("g", self.g_ch)) if c]
+        """Row counts of the ``[dq or q | dkv | g]`` segments of ``in_proj`` (absent ones are left out)."""
+        return [(n, c) for n, c in (("q" if self.q_rank is None else "dq", self.q_ch), ("dkv", self.c_ch), ("g", self.g_ch)) if c]
 
     def _flash_prefill(self, proj, ctx) -> bool:
         import os
 
         return (ctx.fresh_prefill and ctx.min_new >= self.FLASH_PREFILL_MIN_TOKENS and proj.is_cuda
                 and proj.dtype in (torch.bfloat16, torch.float16) and max(self.qk_dim + self.rot_dim, self.v_dim) <= 128
-                and os.environ.get("B200_LATENT_FLASH_PREFILL", "1") == "1" and ops.native_attention_available())
+                and self.softmax_scale > 0.0 and os.environ.get("B200_LATENT_FLASH_PREFILL", "1") == "1" and ops.native_attention_available())
 
-    def forward(self, hidden_states, attention_mask=None, inference_context=None, cache_index=None, **_):
+    def _source_rows(self, ctx, cross_layer):
+        """This step's latents ``[T, r]`` and rotated keys ``[T, n]`` of the layer whose rows this layer shares."""
+        rows = (cross_layer or {}).get(self.kv_source_layer)
+        if rows is not None:
+            return rows
+        if ctx is None:
+            raise RuntimeError(f"layer {self.kv_source_layer} has left no latents for layer {self.layer_number}")
+        c = ctx.step_latents(self.kv_source_layer)
+        return c[:, :self.kv_rank], c[:, self.kv_rank:]
+
+    def forward(self, hidden_states, attention_mask=None, inference_context=None, cache_index=None, cross_layer=None, **_):
         from ..ops import seqmix
         from ..ops.seqmix import HeadPart
         from ..ssm.gated_delta import packed_tokens, unpacked_tokens
         from .mixed_head_attention import dense_pages
 
         s, b = hidden_states.shape[0], hidden_states.shape[1]
-        key = self.layer_number if cache_index is None else cache_index
+        shared = self.kv_source_layer is not None
+        key = self.kv_source_layer if shared else (self.layer_number if cache_index is None else cache_index)
         nh, d, n, dv, r = self.nh, self.qk_dim, self.rot_dim, self.v_dim, self.kv_rank
         proj, _ = self.in_proj(hidden_states)
-        proj = packed_tokens(proj)                                                     # [T, dq | c | k_r | g]
-        T, o0 = proj.shape[0], self.q_rank
-        gate = proj[:, o0 + r + n:] if self.g_ch else None
+        proj = packed_tokens(proj)                                                     # [T, q or dq | c | k_r | g]
+        T, o0 = proj.shape[0], self.q_ch
+        gate = proj[:, o0 + self.c_ch:] if self.g_ch else None
         ctx = inference_context
+        pages = slots = None
         if ctx is not None:
             if ctx.is_static_batching():
                 raise NotImplementedError("latent attention serves through the dynamic (paged) engine")
-            pages, slots, positions = ctx.latent_pages(key, r + n, proj.dtype), ctx.write_slots, ctx.positions
+            slots, positions = ctx.write_slots, ctx.positions
+            if not shared:
+                pages = ctx.latent_pages(key, r + n, proj.dtype)
         else:
             table, tok_req, tok_len = dense_pages(s, b, proj.device)
-            pages, slots, positions = None, None, tok_len.long() - 1
+            positions = tok_len.long() - 1
         flash = ctx is not None and self._flash_prefill(proj, ctx)
-        cq = proj.new_empty(T, 1, o0)
         dense = flash or ctx is None
-        c_out, kr_out = (proj.new_empty(T, 1, r), proj.new_empty(T, 1, n)) if dense else (None, None)
-        c_page, kr_page = (None, None) if pages is None else (pages[:, :r].unsqueeze(1), pages[:, r:].unsqueeze(1))
         rot = dict(turns=self.turns, interleaved=self.interleaved, amplitude=self.amplitude)
-        seqmix.head_rotary([HeadPart(proj[:, :o0].unsqueeze(1), rms=True, weight=self.q_norm_weight, out=cq),
-                            HeadPart(proj[:, o0:o0 + r].unsqueeze(1), rms=True, weight=self.kv_norm_weight, out=c_out,
-                                     pages=c_page),
-                            HeadPart(proj[:, o0 + r:o0 + r + n].unsqueeze(1), out=kr_out, pages=kr_page, **rot)],
-                           positions, self.eps, slots)
-        q, _ = self.linear_q_up_proj(cq[:, 0])
-        q = q.view(T, nh, d + n)
+        q = proj[:, :o0].unflatten(1, (nh, d + n)) if self.q_rank is None else None
+        cq = proj.new_empty(T, 1, o0) if q is None else None
+        q_rot = None if flash else proj.new_empty(T, nh, n)
+        parts, c_out, kr_out = [], None, None
+        if q is None:
+            parts.append(HeadPart(proj[:, :o0].unsqueeze(1), rms=True, weight=self.q_norm_weight, out=cq))
+        elif not flash:
+            parts.append(HeadPart(q[..., d:], out=q_rot, **rot))
+        if not shared:
+            c_out, kr_out = (proj.new_empty(T, 1, r), proj.new_empty(T, 1, n)) if dense else (None, None)
+            c_page, kr_page = (None, None) if pages is None else (pages[:, :r].unsqueeze(1), pages[:, r:].unsqueeze(1))
+            parts += [HeadPart(proj[:, o0:o0 + r].unsqueeze(1), rms=True, weight=self.kv_norm_weight, out=c_out, pages=c_page),
+                      HeadPart(proj[:, o0 + r:o0 + r + n].unsqueeze(1), out=kr_out, pages=kr_page, **rot)]
+        if parts:
+            seqmix.head_rotary(parts, positions, self.eps, slots)
+        if dense and not shared:
+            c_out, kr_out = c_out[:, 0], kr_out[:, 0]
+            if cross_layer is not None:
+                cross_layer[self.layer_number] = (c_out, kr_out)
+        elif dense:
+            c_out, kr_out = self._source_rows(ctx, cross_layer)
+        if q is None:
+            q = self.linear_q_up_proj(cq[:, 0])[0].view(T, nh, d + n)
+            if not flash:
+                seqmix.head_rotary([HeadPart(q[..., d:], out=q_rot, **rot)], positions, self.eps)
         if flash:
             width = 64 if max(d + n, dv) <= 64 else 128
-            k, v = self.linear_k_up_proj(c_out[:, 0])[0].view(T, nh, d), self.linear_v_up_proj(c_out[:, 0])[0].view(T, nh, dv)
+            k, v = self.linear_k_up_proj(c_out)[0].view(T, nh, d), self.linear_v_up_proj(c_out)[0].view(T, nh, dv)
             qp, kp, vp = (proj.new_empty(T, nh, width) for _ in range(3))
-            seqmix.latent_head_assemble(q, k, kr_out[:, 0], v, self.turns, self.interleaved, self.amplitude, positions, qp, kp, vp)
-            cu = ctx.packed.cu_host
-            o = ops.attention_varlen(qp, kp, vp, (cu, cu), None, self.softmax_scale, True, 0.0, False)[..., :dv]
-            o = seqmix.head_gate(o, gate, proj.dtype)
+            seqmix.latent_head_assemble(q, k, kr_out, v, self.turns, self.interleaved, self.amplitude, positions, qp, kp, vp)
+            if self.window or self.sink is not None or self.element_gate:
+                o = ops.window_attention(qp, kp, vp, ctx.packed.cu, ctx.packed.max_len, self.softmax_scale, self.window, self.sink,
+                                         gate if self.element_gate else None, dv).view(T, nh, dv)
+                o = o if self.element_gate else seqmix.head_gate(o, gate, proj.dtype)
+            else:
+                cu = ctx.packed.cu_host
+                o = ops.attention_varlen(qp, kp, vp, (cu, cu), None, self.softmax_scale, True, 0.0, False)[..., :dv]
+                o = seqmix.head_gate(o, gate, proj.dtype)
         else:
-            q_rot = proj.new_empty(T, nh, n)
-            seqmix.head_rotary([HeadPart(q[..., d:], out=q_rot, **rot)], positions, self.eps)
             wk, wv = self.linear_k_up_proj.weight.view(nh, d, r), self.linear_v_up_proj.weight.view(nh, dv, r)
             q_lat = torch.einsum("thd,hdr->thr", q[..., :d], wk)
+            head_gate = None if self.element_gate else gate
             if ctx is not None:
-                o_lat = ctx.attend_latent(key, q_lat, None, self.softmax_scale, q_rot, gate)
+                o_lat = ctx.attend_latent(key, q_lat, None, self.softmax_scale, q_rot, head_gate, self.window, self.sink)
             else:
-                o_lat = seqmix.latent_attention_paged(q_lat, torch.cat([c_out, kr_out], dim=-1)[:, 0], table, tok_req, tok_len, s, self.softmax_scale, 0, q_rot, gate)
+                o_lat = seqmix.latent_attention_paged(q_lat, torch.cat([c_out, kr_out], dim=-1), table, tok_req, tok_len, s, self.softmax_scale,
+                                                      0, q_rot, head_gate, self.window, self.sink)
             o = torch.einsum("thr,hvr->thv", o_lat.to(wv.dtype), wv)
+            if self.element_gate:
+                o = seqmix.head_gate(o, gate, proj.dtype)
         return self.linear_proj(unpacked_tokens(o.reshape(T, nh * dv), s, b))

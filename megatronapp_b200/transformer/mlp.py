@@ -146,6 +146,19 @@ class ClampedGLU:
         return hash((self.limit, self.alpha, self.shift))
 
 
+def gelu_glu(x):
+    """Gated activation over the packed ``[gate | up]`` output of fc1: ``gelu_tanh(gate) * up`` in fp32, one sm_100a kernel
+    (``ops.seqmix.gelu_mul``).  Use as ``activation_func`` with ``gated_linear_unit=True``."""
+    from ..ops import seqmix
+
+    n = x.shape[-1] // 2
+    x2 = x.reshape(-1, 2 * n)
+    return seqmix.gelu_mul(x2[:, :n], x2[:, n:]).view(*x.shape[:-1], n)
+
+
+gelu_glu.fused_glu = True
+
+
 class PolyNorm(torch.nn.Module):
     """Activation with four learned numbers ``coef = (a, b, c, e)``: ``a N(z) + b N(z^2) + c N(z^3) + e``, powers taken element
     by element, ``N`` dividing a token's vector by its root mean square (``eps`` inside the root).  One sm_100a kernel

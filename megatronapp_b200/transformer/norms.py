@@ -130,6 +130,41 @@ class OutputRMSNormAdd(nn.Module):
         return x2.view(shape), y.view(shape)
 
 
+class SquashNorm(nn.Module):
+    """Norm without statistics, element by element: ``tanh(alpha * x) * weight + bias`` with a learned scalar ``alpha`` (Zhu et al.,
+    "Transformers without Normalization").  ``add`` uses it on a sublayer's output: the squashed output times ``mult`` joins the fp32
+    stream and the next norm of the stream comes out of the same kernel (``ops.seqmix.squash_add``)."""
+
+    def __init__(self, config, hidden_size: int, alpha_init: float = 0.5):
+        super().__init__()
+        dtype = config.params_dtype if config is not None else torch.float32
+        dev = "cpu" if (config is None or config.use_cpu_initialization or not torch.cuda.is_available()) \
+            else torch.cuda.current_device()
+        self.hidden_size = hidden_size
+        self.alpha = nn.Parameter(torch.tensor(alpha_init, dtype=dtype, device=dev))
+        self.weight = nn.Parameter(torch.ones(hidden_size, dtype=dtype, device=dev))
+        self.bias = nn.Parameter(torch.zeros(hidden_size, dtype=dtype, device=dev))
+
+    def triple(self):
+        return self.alpha, self.weight, self.bias
+
+    def forward(self, x, x_scale: float = 1.0):
+        """``(x_scale * x, norm(x_scale * x))`` of the fp32 stream ``x``, which is scaled in place."""
+        from ..ops import seqmix
+
+        _, h = seqmix.squash_add(x.view(-1, self.hidden_size), None, None, self.triple(), 0.0, self.weight.dtype, x_scale)
+        return x, h.view(x.shape)
+
+    def add(self, x, out, mult: float = 1.0, next_norm: "SquashNorm" = None):
+        """``x + mult * norm(out)`` (in place) and ``next_norm`` of it (``None`` without one)."""
+        from ..ops import seqmix
+
+        W = self.hidden_size
+        _, h = seqmix.squash_add(x.view(-1, W), out.reshape(-1, W), self.triple(), None if next_norm is None else next_norm.triple(), mult,
+                                 self.weight.dtype)
+        return x, None if h is None else h.view(x.shape)
+
+
 class ScaledPair:
     """Outputs of two mixers that ran side by side on the same input whose result is the weighted sum
     ``scale_a * (a + bias_a) + scale_b * b``; ``StreamConnection`` computes it inside its kernel, in fp32."""
