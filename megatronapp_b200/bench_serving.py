@@ -6,7 +6,9 @@ closest existing model, Lerorax (two mixers side by side on a paged attention an
 beside their like kernels; with ``--serving-design nunosun`` the Nunosun design beside its closest existing model, Domasun
 (sliding-window attention beside a recurrent memory, mixtures of experts), and its kernels beside their like kernels; with
 ``--serving-design nasipel`` the Nasipel design beside its closest existing model, Zikunex (latent attention, recurrent mixers,
-group-limited mixtures of experts), and its kernels beside their like kernels.
+group-limited mixtures of experts), and its kernels beside their like kernels; with ``--serving-design dufitar`` the Dufitar design
+beside its closest existing model, Nasipel (rotary grouped-query attention and rotary latent attention with tcgen05 prompts), and its
+kernels beside their like kernels over as many visible keys.
 
 Two parts, random weights, bf16:
 
@@ -694,6 +696,149 @@ def kernel_numbers_nasipel(s, device):
     return out, roof
 
 
+DUFITAR_WINDOW = 1024
+
+
+def dufitar_config(s):
+    """A Dufitar stack at the sizes of ``s``: latent attention whose heads are three quarters unrotated, two layers of grouped-query
+    attention (a key / value head per four query heads, a quarter of each head turning), latent attention over the first one's
+    latents; every layer with a gated dense feed-forward of the parameter count that a token meets in the mixture of ``s``."""
+    H, d = s["heads"], s["dim"]
+    rot, mask = d // 4, {"size": DUFITAR_WINDOW}
+    ff = {"kind": "dense", "ff": s["expert_ff"] * s["top"]}
+    att = {"heads": H, "kv_heads": max(1, H // 4), "dim": d, "vdim": d, "scale": d ** -0.5, "mask": mask,
+           "rot": {"dims": rot, "base": 10000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    lat = {"heads": H, "dim": d - rot, "rot_dim": rot, "vdim": d, "kv_rank": s["kv_rank"], "scale": d ** -0.5, "mask": mask,
+           "rot": {"base": 10000.0, "dims": rot}}
+    pattern = [("latent_attention", lat), ("attention", att), ("attention", att), ("latent_attention", lat)]
+    layers = []
+    for i in range(s["layers"]):
+        kind, mx = pattern[i % 4]
+        layers.append({"type": kind, "mixer": dict(mx, kv_from=i - 3) if i % 4 == 3 else dict(mx), "mlp": ff})
+    return {"architecture": "Dufitar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0},
+            "residual_mult": 0.5, "layers": layers}
+
+
+def build_dufitar(s, device):
+    from .models.dufitar import DufitarConfig, DufitarModel
+    from .parallel import state as ps
+
+    if not ps.model_parallel_is_initialized():
+        ps.initialize_model_parallel(1, 1)
+    dcfg = DufitarConfig.from_dict(dufitar_config(s))
+    base = dcfg.base_transformer_config(torch.bfloat16, use_cpu_initialization=False)
+    return DufitarModel(dcfg, base).to(device).eval()
+
+
+def kernel_numbers_dufitar(s, device):
+    """The kernels of the Dufitar design and their like kernels: time, achieved bytes/s (or flop/s) and the fraction of the roofline
+    (measured copy bandwidth; for products on the tensor cores the measured cuBLAS rate, on the CUDA cores fp32 FMA).  Windowed
+    attention counts the visible pairs only; the like kernels of the decoding batches hold as many keys as the window shows."""
+    from . import ops
+    from .ops import seqmix
+    from .ops.seqmix import HeadPart
+
+    bench, out, roof = _kernel_bench(device)
+    rn = lambda *sh, dtype=torch.float32: torch.randn(*sh, device=device, dtype=dtype)  # noqa: E731
+    H, d, W, r, w = s["heads"], s["dim"], s["width"], s["kv_rank"], DUFITAR_WINDOW
+    bf = torch.bfloat16
+    G, rot = max(1, H // 4), d // 4
+    # -- decode attention: 64 requests x 2048 cached tokens, the last w of them visible
+    R, L, bs = 64, 2048, 16
+    nblk = R * L // bs
+    table = torch.randperm(nblk, device=device).to(torch.int32).view(R, L // bs)
+    req = torch.arange(R, dtype=torch.int32, device=device)
+    lens, lens_w = (torch.full((R,), n, dtype=torch.int32, device=device) for n in (L, w))
+    kc, vc, q = rn(nblk * bs, G, d, dtype=bf), rn(nblk * bs, G, d, dtype=bf), rn(R, H, d, dtype=bf)
+    bench("window_attention_paged.decode", lambda: seqmix.window_attention_paged(q, kc, vc, table, req, lens, bs, d ** -0.5, w, max_len=L),
+          R * w * G * d * 4, flops=R * w * H * d * 4, like="sigmoid_attention_paged.decode")
+    turns = seqmix.rotary_turns(d, 10000.0, device=device)[0]
+    hb = torch.randn(H, device=device) - 4.0
+    bench("sigmoid_attention_paged.decode", lambda: seqmix.sigmoid_attention_paged(q, kc, vc, table, req, lens_w, bs, d ** -0.5, 30.0, hb, turns,
+                                                                                   False, w), R * w * G * d * 4, flops=R * w * H * d * 4)
+    cache = rn(nblk * bs, r + rot, dtype=bf)
+    ql, qr, gate, sink = rn(R, H, r, dtype=bf), rn(R, H, rot, dtype=bf), rn(R, H, dtype=bf), rn(H, dtype=bf)
+    bench("latent_attention_paged.decode (window, sink)",
+          lambda: seqmix.latent_attention_paged(ql, cache, table, req, lens, bs, 0.05, L, qr, None, w, sink),
+          R * w * (r + rot) * 2, flops=R * w * H * (2 * r + rot) * 2, like="latent_attention_paged.decode (gate)")
+    bench("latent_attention_paged.decode (gate)", lambda: seqmix.latent_attention_paged(ql, cache, table, req, lens_w, bs, 0.05, w, qr, gate),
+          R * w * (r + rot) * 2, flops=R * w * H * (2 * r + rot) * 2)
+    # -- prompts: 4 x 2048 tokens
+    n = 2048
+    T = 4 * n
+    cu = torch.tensor([0, n, 2 * n, 3 * n, T], dtype=torch.int32, device=device)
+    pos = torch.arange(n, device=device).repeat(4)
+    pairs, pairs_w = n * (n + 1) / 2, w * (w + 1) / 2 + (n - w) * w
+    q4, k4, v4 = rn(T, H, d, dtype=bf), rn(T, G, d, dtype=bf), rn(T, G, d, dtype=bf)
+    kh, vh, ge = rn(T, H, d, dtype=bf), rn(T, H, d, dtype=bf), rn(T, H * d, dtype=bf)
+    tab = rn(T, d // 2, 2)
+    bench("window_attention (tcgen05).prefill", lambda: ops.window_attention(q4, k4, v4, cu, n, d ** -0.5, w),
+          T * (H * 2 + G * 2) * d * 2, flops=4 * pairs_w * H * d * 4, like="sigmoid_attention (tcgen05).prefill", tensor=True)
+    bench("window_attention (tcgen05).prefill (sink, gate, keys per head)",
+          lambda: ops.window_attention(q4, kh, vh, cu, n, d ** -0.5, w, sink, ge),
+          T * H * 5 * d * 2, flops=4 * pairs_w * H * d * 4, like="sigmoid_attention (tcgen05).prefill", tensor=True)
+    bench("window_attention (tcgen05).prefill (no window)", lambda: ops.window_attention(q4, k4, v4, cu, n, d ** -0.5),
+          T * (H * 2 + G * 2) * d * 2, flops=4 * pairs * H * d * 4, like="attn_fwd (tcgen05).prefill", tensor=True)
+    bench("sigmoid_attention (tcgen05).prefill", lambda: ops.sigmoid_attention(q4, k4, v4, cu, n, d ** -0.5, 30.0, hb, tab, False, d),
+          T * (H * 2 + G * 2) * d * 2, flops=4 * pairs * H * d * 4, tensor=True)
+    cuh = [0, n, 2 * n, 3 * n, T]
+    bench("attn_fwd (tcgen05).prefill", lambda: ops.attention_varlen(q4, k4, v4, (cuh, cuh), None, d ** -0.5, True, 0.0, False),
+          T * (H * 2 + G * 2) * d * 2, flops=4 * pairs * H * d * 4, tensor=True)
+    table1 = torch.randperm(n // bs, device=device).to(torch.int32).view(1, -1)
+    req1 = torch.zeros(n, dtype=torch.int32, device=device)
+    len1 = torch.arange(1, n + 1, dtype=torch.int32, device=device)
+    bench("window_attention_paged.prefill (1 x 2048)",
+          lambda: seqmix.window_attention_paged(q4[:n], kc, vc, table1, req1, len1, bs, d ** -0.5, w),
+          n * (H * 2 + G * 2) * d * 2, flops=pairs_w * H * d * 4, like="sigmoid_attention_paged.prefill (1 x 2048)")
+    bench("sigmoid_attention_paged.prefill (1 x 2048)",
+          lambda: seqmix.sigmoid_attention_paged(q4[:n], kc, vc, table1, req1, len1, bs, d ** -0.5, 30.0, hb, turns),
+          n * (H * 2 + G * 2) * d * 2, flops=pairs * H * d * 4)
+    q1, qr1, g1 = rn(n, H, r, dtype=bf), rn(n, H, rot, dtype=bf), rn(n, H, dtype=bf)
+    bench("latent_attention_paged.prefill (1 x 2048, window, sink)",
+          lambda: seqmix.latent_attention_paged(q1, cache, table1, req1, len1, bs, 0.05, n, qr1, None, w, sink),
+          n * (r + rot) * 2 + n * H * r * 6, flops=pairs_w * H * (2 * r + rot) * 2, like="latent_attention_paged.prefill (1 x 2048, gate)")
+    bench("latent_attention_paged.prefill (1 x 2048, gate)",
+          lambda: seqmix.latent_attention_paged(q1, cache, table1, req1, len1, bs, 0.05, n, qr1, g1),
+          n * (r + rot) * 2 + n * H * r * 6, flops=pairs * H * (2 * r + rot) * 2)
+    # -- additions and norms, activation, rotations, gates over 8192 tokens
+    x = rn(T, W)
+    a, b, ga, gb = (rn(T, W, dtype=bf) for _ in range(4))
+    one, al = torch.ones(W, device=device, dtype=bf), torch.tensor(0.5, device=device, dtype=bf)
+    bench("squash_add (addend, two norms)", lambda: seqmix.squash_add(x, a, (al, one, one), (al, one, one), 0.5, bf), T * W * (4 + 4 + 2 + 2),
+          like="gated_add_norm (two gated addends, two norms)")
+    bench("gated_add_norm (two gated addends, two norms)", lambda: seqmix.gated_add_norm(x, a, ga, one, b, gb, one, one, one, 1e-5, bf),
+          T * W * (4 + 4 + 2 * 4 + 2 * 2))
+    ff = s["expert_ff"] * s["top"]
+    gu = rn(T, 2 * ff, dtype=bf)
+    bench("gelu_mul", lambda: seqmix.gelu_mul(gu[:, :ff], gu[:, ff:]), T * ff * 6, like="swiglu")
+    bench("swiglu", lambda: ops.swiglu(gu), T * ff * 6)
+    proj = rn(T, (H + 2 * G) * d, dtype=bf)
+    qo, ko, vo = rn(T, H, d, dtype=bf), rn(T, G, d, dtype=bf), rn(T, G, d, dtype=bf)
+    slots = torch.randperm(nblk * bs, device=device)[:T]
+    qv, kv_, vv = (proj[:, i0 * d:(i0 + h) * d].unflatten(1, (h, d)) for i0, h in ((0, H), (H, G), (H + G, G)))
+    tr, amp = seqmix.rotary_turns(rot, 10000.0, {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}, device)
+    nbytes = T * (H + 2 * G) * d * 4 + T * 2 * G * d * 2
+    kw = dict(turns=tr, interleaved=True, amplitude=amp)
+    bench("head_rotary (a part of q, k; pages)",
+          lambda: seqmix.head_rotary([HeadPart(qv, out=qo, **kw), HeadPart(kv_, out=ko, pages=kc, **kw), HeadPart(vv, out=vo, pages=vc)], pos, 0.0,
+                                     slots), nbytes, like="head_rotary (q, k, v; norm; pages)")
+    kn = dict(turns=turns, rms=True)
+    bench("head_rotary (q, k, v; norm; pages)",
+          lambda: seqmix.head_rotary([HeadPart(qv, out=qo, **kn), HeadPart(kv_, out=ko, pages=kc, **kn), HeadPart(vv, turns, out=vo, pages=vc)], pos,
+                                     1e-5, slots), nbytes)
+    lp = rn(T, H * d + r + rot, dtype=bf)
+    q_all, k_n, k_r = lp[:, :H * d].unflatten(1, (H, d)), rn(T, H, d - rot, dtype=bf), rn(T, rot, dtype=bf)
+    oo = [rn(T, H, d, dtype=bf) for _ in range(3)]
+    bench("latent_head_assemble (strided q)", lambda: seqmix.latent_head_assemble(q_all, k_n, k_r, vh, tr, True, 1.0, pos, *oo),
+          T * H * d * (2 * 6), like="latent_head_assemble")
+    qc = q_all.contiguous()
+    bench("latent_head_assemble", lambda: seqmix.latent_head_assemble(qc, k_n, k_r, vh, tr, True, 1.0, pos, *oo), T * H * d * (2 * 6))
+    gh = rn(T, H, dtype=bf)
+    bench("head_gate (elementwise)", lambda: seqmix.head_gate(oo[0], ge, bf), T * H * d * 6, like="head_gate")
+    bench("head_gate", lambda: seqmix.head_gate(oo[0], gh, bf), T * H * d * 4)
+    return out, roof
+
+
 def kernel_numbers(s, device):
     """Every new kernel alone and its like kernel: time, achieved bytes/s (or flop/s) and the fraction of the roofline."""
     from . import ops
@@ -822,7 +967,8 @@ def run(args):
              "lerorax": (("lerorax", build_lerorax), ("zikunex", build_zikunex)),
              "domasun": (("domasun", build_domasun), ("lerorax", build_lerorax)),
              "nunosun": (("nunosun", build_nunosun), ("domasun", build_domasun)),
-             "nasipel": (("nasipel", build_nasipel), ("zikunex", build_zikunex))}[design]
+             "nasipel": (("nasipel", build_nasipel), ("zikunex", build_zikunex)),
+             "dufitar": (("dufitar", build_dufitar), ("nasipel", build_nasipel))}[design]
     with torch.no_grad():
         for name, build in pairs:
             t0 = time.time()
@@ -835,7 +981,7 @@ def run(args):
             torch.cuda.empty_cache()
         if not getattr(args, "serving_models_only", False):
             fn = {"zikunex": kernel_numbers, "lerorax": kernel_numbers_lerorax, "domasun": kernel_numbers_domasun,
-                  "nunosun": kernel_numbers_nunosun, "nasipel": kernel_numbers_nasipel}[design]
+                  "nunosun": kernel_numbers_nunosun, "nasipel": kernel_numbers_nasipel, "dufitar": kernel_numbers_dufitar}[design]
             res["kernels"], res["roofline"] = fn(s, dev)
     print(json.dumps(res), flush=True)
     return res
