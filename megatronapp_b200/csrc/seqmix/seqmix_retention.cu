@@ -223,6 +223,11 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z,
   }
 }
 
+// z / 2 (1 + tanh u) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3): no cancellation for negative z, one exponential
+__device__ __forceinline__ float gelu_tanh(float z) {
+  return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
+
 template <typename T>
 __global__ void gelu_mul_kernel(const T* __restrict__ g, int64_t ldg, const T* __restrict__ e, int64_t lde, T* __restrict__ y,
                                 int64_t rows, int cols) {
@@ -230,9 +235,7 @@ __global__ void gelu_mul_kernel(const T* __restrict__ g, int64_t ldg, const T* _
   if (idx >= rows * cols) return;
   const int64_t r = idx / cols;
   const int c = static_cast<int>(idx - r * cols);
-  const float zv = ld(g + r * ldg + c);
-  const float act = 0.5f * zv * (1.0f + tanhf(0.7978845608028654f * (zv + 0.044715f * zv * zv * zv)));
-  st(y + idx, act * ld(e + r * lde + c));
+  st(y + idx, gelu_tanh(ld(g + r * ldg + c)) * ld(e + r * lde + c));
 }
 
 // four columns per thread, a row per blockIdx.y step (cols a multiple of 4, aligned rows)
@@ -255,7 +258,6 @@ template <> struct Quad<__nv_bfloat16> {
     *reinterpret_cast<uint2*>(p) = r;
   }
 };
-__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 
 template <typename T>
 __global__ void __launch_bounds__(256) gelu_mul_vec_kernel(const T* __restrict__ g, int64_t ldg, const T* __restrict__ e, int64_t lde,
