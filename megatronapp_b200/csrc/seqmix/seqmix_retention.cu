@@ -225,7 +225,7 @@ __global__ void __launch_bounds__(256) poly_norm_kernel(const T* __restrict__ z,
 
 // z / 2 (1 + tanh u) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3): no cancellation for negative z, one exponential
 __device__ __forceinline__ float gelu_tanh(float z) {
-  return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+  return __fdividef(z, 1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 template <typename T>
